@@ -130,11 +130,14 @@ class RunEntry:
     `copy`: a layer that runs several times with the same weights but with keys and
     state of its own each time names a different copy in each of its entries (a
     reader reads the copy of the same number).  `add`: (name of one of the model's
-    `vectors`, row): that row is added to the residual rows before the layer runs."""
+    `vectors`, row): that row is added to the residual rows before the layer runs.
+    `add_embedding`: the embedding's output (the rows as they were before the first layer)
+    is added to them before that."""
     layer: int
     cache_of: Optional[int] = None
     copy: int = 0
     add: Optional[Tuple[str, int]] = None
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

@@ -58,7 +58,16 @@ struct AttnParams {
     int gate_stride;
     int gate_per_head;           // 1: a gate row holds one logit per head instead
     float out_scale;
+    int value_dim;               // size of a value (a key's unless the kernel is the DV form)
+    int chunked;                 // 1: `window` is the size of chunks counted from position 0; a row
+                                 // sees the keys of its own chunk up to itself
 };
+
+// The first key that a row at position `pos` sees behind the kept first tokens.
+__device__ __forceinline__ int first_key(const AttnParams& p, int pos) {
+    if (p.window <= 0) return 0;
+    return p.chunked ? pos - pos % p.window : max(0, pos - p.window + 1);
+}
 
 __device__ __forceinline__ uint32_t smem_u32(const void* p) {
     return (uint32_t)__cvta_generic_to_shared(p);
@@ -110,7 +119,8 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 // kernel's life and worked out once; per tile only the page lookup remains (a
 // shift and a mask when the page size is a power of two).  Keys at or beyond
 // `key_end` are zero-filled.
-template <int HD_MAX, int NT, int TILE>
+// DV: values of a size of their own: their pieces are worked out apart from the keys'.
+template <int HD_MAX, int NT, int TILE, bool DV = false>
 struct KvLoader {
     static constexpr int ITEMS = (TILE * (HD_MAX / 8) + NT - 1) / NT;
     int row[ITEMS];          // key row inside the tile, or -1
@@ -118,6 +128,25 @@ struct KvLoader {
     int sdst[ITEMS];         // byte offset of the piece inside a shared-memory tile
     size_t page_elems;       // elements of one page (all KV heads)
     int page_shift;          // log2(page_tokens), or -1 if not a power of two
+    int dim;                 // features of a row
+
+    // the rows of one operand alone (DV form): `dim_` features a row
+    __device__ __forceinline__ void init_one(const AttnParams& p, int kv_head, int pitch, int tid, int dim_) {
+        dim = dim_;
+        const int chunks_per_row = dim >> 3;
+        const int total = TILE * chunks_per_row;
+#pragma unroll
+        for (int u = 0; u < ITEMS; ++u) {
+            const int i = tid + u * NT;
+            const int r = i / chunks_per_row;
+            const int col = (i - r * chunks_per_row) * 8;
+            row[u] = i < total ? r : -1;
+            base[u] = kv_head * p.page_tokens * dim + col;
+            sdst[u] = (r * pitch + col) * 2;
+        }
+        page_elems = (size_t)p.n_kv_heads * p.page_tokens * dim;
+        page_shift = (p.page_tokens & (p.page_tokens - 1)) == 0 ? 31 - __clz(p.page_tokens) : -1;
+    }
 
     __device__ __forceinline__ void init(const AttnParams& p, int kv_head, int pitch, int tid) {
         const int chunks_per_row = p.head_dim >> 3;
@@ -131,6 +160,7 @@ struct KvLoader {
             base[u] = kv_head * p.page_tokens * p.head_dim + col;
             sdst[u] = (r * pitch + col) * 2;
         }
+        dim = p.head_dim;
         page_elems = (size_t)p.n_kv_heads * p.page_tokens * p.head_dim;
         page_shift = (p.page_tokens & (p.page_tokens - 1)) == 0 ? 31 - __clz(p.page_tokens) : -1;
     }
@@ -138,7 +168,14 @@ struct KvLoader {
     __device__ __forceinline__ void load(const AttnParams& p, const int* table, int key0,
                                          int key_end, __nv_bfloat16* k_smem,
                                          __nv_bfloat16* v_smem) const {
-        const uint32_t ks = smem_u32(k_smem), vs = smem_u32(v_smem);
+        copy(p, table, key0, key_end, p.k_cache, k_smem, p.v_cache, v_smem);
+    }
+
+    // DV: one operand's tile (src2 is not read)
+    __device__ __forceinline__ void copy(const AttnParams& p, const int* table, int key0, int key_end,
+                                         const __nv_bfloat16* src, __nv_bfloat16* dst,
+                                         const __nv_bfloat16* src2, __nv_bfloat16* dst2) const {
+        const uint32_t ks = smem_u32(dst), vs = smem_u32(DV ? dst : dst2);
         // in batches of four pieces: first the block-table lookups (loads that may
         // miss), then the copies, so that the lookups' latencies overlap
 #pragma unroll
@@ -169,7 +206,7 @@ struct KvLoader {
                         valid[v] = page >= 0;
                         if (valid[v])
                             off[v] = (size_t)page * page_elems +
-                                     (size_t)(base[u] + slot * p.head_dim);
+                                     (size_t)(base[u] + slot * (DV ? dim : p.head_dim));
                     }
                 }
             }
@@ -179,9 +216,10 @@ struct KvLoader {
                 if (u < ITEMS && row[u] >= 0) {
                     const int bytes = valid[v] ? 16 : 0;     // 0: zero-filled
                     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(ks + sdst[u]),
-                                 "l"(p.k_cache + off[v]), "r"(bytes) : "memory");
-                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vs + sdst[u]),
-                                 "l"(p.v_cache + off[v]), "r"(bytes) : "memory");
+                                 "l"(src + off[v]), "r"(bytes) : "memory");
+                    if (!DV)
+                        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(vs + sdst[u]),
+                                     "l"(src2 + off[v]), "r"(bytes) : "memory");
                 }
             }
         }
@@ -227,7 +265,7 @@ struct QFrags {
 // Rows g = lane / 4 and g + 8.  `masked`: some key of the tile may lie outside a
 // row's range (after its position, before its window, or past the end); when
 // the caller knows that none does, the per-element tests are skipped.
-template <int HD_MAX, int NK, bool EXACT, bool EXT = false>
+template <int HD_MAX, int NK, bool EXACT, bool EXT = false, bool DV = false>
 __device__ __forceinline__ void attend_tile(const AttnParams& p, const QFrags<HD_MAX>& q,
                                             const __nv_bfloat16* k_smem,
                                             const __nv_bfloat16* v_smem, int pitch_, bool masked,
@@ -240,6 +278,7 @@ __device__ __forceinline__ void attend_tile(const AttnParams& p, const QFrags<HD
     // EXACT: the head size is HD_MAX itself, so the loop bounds and the row pitch are
     // constants and the address arithmetic folds away
     const int hd = EXACT ? HD_MAX : p.head_dim;
+    const int vd = DV ? p.value_dim : hd;
     const int pitch = EXACT ? HD_MAX + 8 : pitch_;
     const int mat = lane >> 3;
     float s[NK / 8][4];
@@ -334,7 +373,7 @@ __device__ __forceinline__ void attend_tile(const AttnParams& p, const QFrags<HD
         a[3] = pack_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3]);
 #pragma unroll
         for (int n = 0; n < HD_MAX / 8; n += 2) {
-            if (n * 8 < hd) {
+            if (n * 8 < vd) {
                 uint32_t b[4];
                 ldmatrix_x4_trans(b, v_lane + kk * 16 * pitch + n * 8);
                 mma_bf16(o[n], a, b[0], b[1]);
@@ -372,12 +411,14 @@ __device__ __forceinline__ void load_q_rows(const AttnParams& p, int row_base, i
 // SPLIT (with EXT, requests of at most 64 packed rows): block x takes one of n_chunks equal
 // shares of the row tile's list of key tiles and leaves its running maximum, sum and
 // unnormalised result in p.partial; `attention_merge_kernel` adds the shares.
-template <int HD_MAX, bool EXACT, bool EXT = false, bool SPLIT = false>
+// DV (with EXT): keys of head_dim, values of value_dim features; both lie in rows of one pitch.
+template <int HD_MAX, bool EXACT, bool EXT = false, bool SPLIT = false, bool DV = false>
 __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p) {
     cb_pdl_trigger();
     cb_pdl_wait();
     extern __shared__ __align__(16) uint8_t smem_raw[];
-    const int pitch = EXACT ? HD_MAX + 8 : p.head_dim + 8;
+    const int pitch = EXACT ? HD_MAX + 8 : (DV ? max(p.head_dim, p.value_dim) : p.head_dim) + 8;
+    const int od = DV ? p.value_dim : p.head_dim;            // features of a head's result
     __nv_bfloat16* q_smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);
     __nv_bfloat16* kv_smem = q_smem + 64 * pitch;      // [2 stages][K, V][64][pitch]
     const int req = blockIdx.z, kv_head = blockIdx.y;
@@ -399,7 +440,7 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
     const int last_row = min(n_rows - 1, qt * 64 + 63);
     const int max_pos = first_pos + last_row / n_rep;
     const int min_pos = first_pos + (qt * 64) / n_rep;
-    int key_lo = p.window > 0 ? max(0, min_pos - p.window + 1) : 0;
+    int key_lo = EXT ? first_key(p, min_pos) : p.window > 0 ? max(0, min_pos - p.window + 1) : 0;
     key_lo = key_lo / TILE_KEYS * TILE_KEYS;
     const int key_end = max_pos + 1;
     // EXT: the tiles that hold the kept first tokens come first, if the window has left them
@@ -412,15 +453,15 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
     const int row_a = qt * 64 + warp * 16 + g, row_b = row_a + 8;
     const int pos_a = row_a < n_rows ? first_pos + row_a / n_rep : -1;
     const int pos_b = row_b < n_rows ? first_pos + row_b / n_rep : -1;
-    const int lo_a = p.window > 0 ? max(0, pos_a - p.window + 1) : 0;
-    const int lo_b = p.window > 0 ? max(0, pos_b - p.window + 1) : 0;
+    const int lo_a = EXT ? first_key(p, pos_a) : p.window > 0 ? max(0, pos_a - p.window + 1) : 0;
+    const int lo_b = EXT ? first_key(p, pos_b) : p.window > 0 ? max(0, pos_b - p.window + 1) : 0;
     const int warp_last_row = min(n_rows - 1, qt * 64 + warp * 16 + 15);
     const int warp_max_pos = qt * 64 + warp * 16 < n_rows ? first_pos + warp_last_row / n_rep : -1;
     // interior tiles: all 16 rows of the warp exist, and the tile lies before the
     // lowest position and inside the latest window of the warp's rows
     const bool warp_full = qt * 64 + warp * 16 + 15 < n_rows;
     const int warp_min_pos = warp_full ? first_pos + (qt * 64 + warp * 16) / n_rep : -1;
-    const int warp_max_lo = p.window > 0 ? max(0, warp_max_pos - p.window + 1) : 0;
+    const int warp_max_lo = EXT ? first_key(p, warp_max_pos) : p.window > 0 ? max(0, warp_max_pos - p.window + 1) : 0;
     QFrags<HD_MAX> qf;
 
     float o[HD_MAX / 8][4];
@@ -429,14 +470,27 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
     float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
 
     const int stage_elems = 2 * TILE_KEYS * pitch;
-    KvLoader<HD_MAX, 128, TILE_KEYS> loader;
-    loader.init(p, kv_head, pitch, threadIdx.x);
+    KvLoader<HD_MAX, 128, TILE_KEYS, DV> loader, loader_v;
+    if (DV) {
+        loader.init_one(p, kv_head, pitch, threadIdx.x, p.head_dim);
+        loader_v.init_one(p, kv_head, pitch, threadIdx.x, p.value_dim);
+    } else {
+        loader.init(p, kv_head, pitch, threadIdx.x);
+    }
+    auto load_tile = [&](int key0, __nv_bfloat16* ks) {
+        if (DV) {
+            loader.copy(p, table, key0, key_end, p.k_cache, ks, nullptr, nullptr);
+            loader_v.copy(p, table, key0, key_end, p.v_cache, ks + TILE_KEYS * pitch, nullptr, nullptr);
+        } else {
+            loader.load(p, table, key0, key_end, ks, ks + TILE_KEYS * pitch);
+        }
+    };
     // SPLIT: this block's share of the tiles
     const int per_chunk = SPLIT ? (n_tiles + p.n_chunks - 1) / p.n_chunks : n_tiles;
     const int tile_begin = SPLIT ? min(n_tiles, (int)blockIdx.x * per_chunk) : 0;
     const int tile_end = SPLIT ? min(n_tiles, tile_begin + per_chunk) : n_tiles;
     if (tile_begin < tile_end)
-        loader.load(p, table, tile_key0(tile_begin), key_end, kv_smem, kv_smem + TILE_KEYS * pitch);
+        load_tile(tile_key0(tile_begin), kv_smem);
     cp_async_commit();
     if (SPLIT && tile_begin >= tile_end) {
         __syncthreads();
@@ -446,7 +500,7 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
         const int st = (i - tile_begin) & 1;
         if (i + 1 < tile_end) {
             __nv_bfloat16* nxt = kv_smem + (st ^ 1) * stage_elems;
-            loader.load(p, table, tile_key0(i + 1), key_end, nxt, nxt + TILE_KEYS * pitch);
+            load_tile(tile_key0(i + 1), nxt);
             cp_async_commit();
             cp_async_wait<1>();
         } else {
@@ -460,7 +514,7 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
             // no test per element if every key of the tile is inside every row's range
             const bool interior = key0 + TILE_KEYS - 1 <= warp_min_pos && key0 >= warp_max_lo &&
                                   i >= keep_tiles;
-            attend_tile<HD_MAX, TILE_KEYS, EXACT, EXT>(p, qf, ks, ks + TILE_KEYS * pitch, pitch, !interior,
+            attend_tile<HD_MAX, TILE_KEYS, EXACT, EXT, DV>(p, qf, ks, ks + TILE_KEYS * pitch, pitch, !interior,
                                                   key0, pos_a, pos_b, lo_a, lo_b, key_end, o, m_a,
                                                   m_b, l_a, l_b);
         }
@@ -474,25 +528,25 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
         // rows of the partials: [request][kv head][chunk][packed row][head_dim + 2]
         const int max_rows = p.chunk_keys;          // the launch's largest count of packed rows
         float* base = p.partial + ((((size_t)req * p.n_kv_heads + kv_head) * p.n_chunks + blockIdx.x) *
-                                   max_rows) * (p.head_dim + 2);
+                                   max_rows) * (od + 2);
 #pragma unroll
         for (int n = 0; n < HD_MAX / 8; ++n) {
-            if (n * 8 < p.head_dim) {
+            if (n * 8 < od) {
                 const int col = n * 8 + 2 * t;
                 if (row_a < n_rows)
-                    *reinterpret_cast<float2*>(base + (size_t)row_a * (p.head_dim + 2) + col) =
+                    *reinterpret_cast<float2*>(base + (size_t)row_a * (od + 2) + col) =
                         make_float2(o[n][0], o[n][1]);
                 if (row_b < n_rows)
-                    *reinterpret_cast<float2*>(base + (size_t)row_b * (p.head_dim + 2) + col) =
+                    *reinterpret_cast<float2*>(base + (size_t)row_b * (od + 2) + col) =
                         make_float2(o[n][2], o[n][3]);
             }
         }
         if (t == 0) {
             if (row_a < n_rows)
-                *reinterpret_cast<float2*>(base + (size_t)row_a * (p.head_dim + 2) + p.head_dim) =
+                *reinterpret_cast<float2*>(base + (size_t)row_a * (od + 2) + od) =
                     make_float2(m_a, l_a);
             if (row_b < n_rows)
-                *reinterpret_cast<float2*>(base + (size_t)row_b * (p.head_dim + 2) + p.head_dim) =
+                *reinterpret_cast<float2*>(base + (size_t)row_b * (od + 2) + od) =
                     make_float2(m_b, l_b);
         }
         return;
@@ -519,7 +573,7 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
     }
 #pragma unroll
     for (int n = 0; n < HD_MAX / 8; ++n) {
-        if (n * 8 < p.head_dim) {
+        if (n * 8 < od) {
             const int col = n * 8 + 2 * t;
             if (row_a < n_rows) {
                 const int tok = row_base + row_a / n_rep, head = kv_head * n_rep + row_a % n_rep;
@@ -531,12 +585,12 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
                     y *= g;
                 } else if (EXT && p.gate != nullptr) {
                     const __nv_bfloat162 gt = *reinterpret_cast<const __nv_bfloat162*>(
-                        p.gate + (size_t)tok * p.gate_stride + (size_t)head * p.head_dim + col);
+                        p.gate + (size_t)tok * p.gate_stride + (size_t)head * od + col);
                     x *= 1.0f / (1.0f + __expf(-__bfloat162float(gt.x)));
                     y *= 1.0f / (1.0f + __expf(-__bfloat162float(gt.y)));
                 }
                 *reinterpret_cast<uint32_t*>(p.out + (size_t)tok * p.out_stride +
-                                             (size_t)head * p.head_dim + col) = pack_bf16(x, y);
+                                             (size_t)head * od + col) = pack_bf16(x, y);
             }
             if (row_b < n_rows) {
                 const int tok = row_base + row_b / n_rep, head = kv_head * n_rep + row_b % n_rep;
@@ -548,12 +602,12 @@ __global__ void __launch_bounds__(128) attention_tiles_kernel(const AttnParams p
                     y *= g;
                 } else if (EXT && p.gate != nullptr) {
                     const __nv_bfloat162 gt = *reinterpret_cast<const __nv_bfloat162*>(
-                        p.gate + (size_t)tok * p.gate_stride + (size_t)head * p.head_dim + col);
+                        p.gate + (size_t)tok * p.gate_stride + (size_t)head * od + col);
                     x *= 1.0f / (1.0f + __expf(-__bfloat162float(gt.x)));
                     y *= 1.0f / (1.0f + __expf(-__bfloat162float(gt.y)));
                 }
                 *reinterpret_cast<uint32_t*>(p.out + (size_t)tok * p.out_stride +
-                                             (size_t)head * p.head_dim + col) = pack_bf16(x, y);
+                                             (size_t)head * od + col) = pack_bf16(x, y);
             }
         }
     }
@@ -814,24 +868,26 @@ __global__ void __launch_bounds__(128) attention_split_kernel(const AttnParams p
     }
 }
 
-template <int HD_MAX, bool EXACT, bool EXT = false>
+template <int HD_MAX, bool EXACT, bool EXT = false, bool DV = false>
 int launch_tiles_as(const AttnParams& p, int n_requests, int max_q_tiles, cudaStream_t s) {
-    const int pitch = p.head_dim + 8;
+    const int pitch = (DV && p.value_dim > p.head_dim ? p.value_dim : p.head_dim) + 8;
     const int smem = (64 + 4 * TILE_KEYS) * pitch * 2;
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tiles_kernel<HD_MAX, EXACT, EXT>,
+        cudaError_t e = cudaFuncSetAttribute(attention_tiles_kernel<HD_MAX, EXACT, EXT, false, DV>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(max_q_tiles, p.n_kv_heads, n_requests);
-    cb_launch(attention_tiles_kernel<HD_MAX, EXACT, EXT>, dim3(grid), dim3(128), smem, s, p);
+    cb_launch(attention_tiles_kernel<HD_MAX, EXACT, EXT, false, DV>, dim3(grid), dim3(128), smem, s, p);
     return cb_last_error();
 }
 
 template <int HD_MAX, bool EXT = false>
 int launch_tiles(const AttnParams& p, int n_requests, int max_q_tiles, cudaStream_t s) {
+    if constexpr (EXT)
+        if (p.value_dim != p.head_dim) return launch_tiles_as<HD_MAX, false, true, true>(p, n_requests, max_q_tiles, s);
     return p.head_dim == HD_MAX ? launch_tiles_as<HD_MAX, true, EXT>(p, n_requests, max_q_tiles, s)
                                 : launch_tiles_as<HD_MAX, false, EXT>(p, n_requests, max_q_tiles, s);
 }
@@ -847,7 +903,7 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const AttnParams p
     const int row_base = p.req_row_start[req];
     const int n_rows = (p.req_row_start[req + 1] - row_base) * n_rep;
     if (row >= n_rows) return;
-    const int hd = p.head_dim, stride = hd + 2;
+    const int hd = p.value_dim, stride = hd + 2;
     const float* base = p.partial + (((size_t)req * p.n_kv_heads + kv_head) * p.n_chunks * max_rows + row) * stride;
     const size_t chunk_stride = (size_t)max_rows * stride;
     // lane c holds share c's maximum and sum (at most 32 shares)
@@ -891,18 +947,18 @@ __global__ void __launch_bounds__(128) attention_merge_kernel(const AttnParams p
     }
 }
 
-template <int HD_MAX, bool EXACT>
+template <int HD_MAX, bool EXACT, bool DV = false>
 int launch_tiles_split_as(const AttnParams& p, int n_requests, int max_rows, cudaStream_t s) {
-    const int pitch = p.head_dim + 8;
+    const int pitch = (DV && p.value_dim > p.head_dim ? p.value_dim : p.head_dim) + 8;
     const int smem = (64 + 4 * TILE_KEYS) * pitch * 2;
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_tiles_kernel<HD_MAX, EXACT, true, true>,
+        cudaError_t e = cudaFuncSetAttribute(attention_tiles_kernel<HD_MAX, EXACT, true, true, DV>,
                                              cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    cb_launch(attention_tiles_kernel<HD_MAX, EXACT, true, true>, dim3(p.n_chunks, p.n_kv_heads, n_requests),
+    cb_launch(attention_tiles_kernel<HD_MAX, EXACT, true, true, DV>, dim3(p.n_chunks, p.n_kv_heads, n_requests),
               dim3(128), smem, s, p);
     cb_launch(attention_merge_kernel, dim3((max_rows + 3) / 4, p.n_kv_heads, n_requests), dim3(128), 0, s,
               p, max_rows);
@@ -911,6 +967,7 @@ int launch_tiles_split_as(const AttnParams& p, int n_requests, int max_rows, cud
 
 template <int HD_MAX>
 int launch_tiles_split(const AttnParams& p, int n_requests, int max_rows, cudaStream_t s) {
+    if (p.value_dim != p.head_dim) return launch_tiles_split_as<HD_MAX, false, true>(p, n_requests, max_rows, s);
     return p.head_dim == HD_MAX ? launch_tiles_split_as<HD_MAX, true>(p, n_requests, max_rows, s)
                                 : launch_tiles_split_as<HD_MAX, false>(p, n_requests, max_rows, s);
 }
@@ -1002,6 +1059,8 @@ CB_EXPORT int cb_attention_mma(const void* qkv, int qkv_stride, void* out, int o
     p.gate_stride = 0;
     p.gate_per_head = 0;
     p.out_scale = 1.0f;
+    p.value_dim = head_dim;
+    p.chunked = 0;
     p.partial = partial;
     p.n_chunks = n_chunks;
     p.chunk_keys = chunk_keys > 0 ? chunk_keys : SPLIT_KEYS;
@@ -1037,19 +1096,19 @@ CB_EXPORT int cb_attention_mma(const void* qkv, int qkv_stride, void* out, int o
 // ([n_heads], may be null) join each head's denominator as exp(sink); the result is multiplied
 // by sigmoid(gate) (rows laid out like `out`, or one logit per head with gate_per_head; may be
 // null) and by out_scale.  q: rows of
-// n_heads * head_dim at q_stride.  Keys and values have the same size.  n_chunks > 1 (requests
+// n_heads * head_dim at q_stride.  chunked: `window` is a chunk's size instead (first_key).  n_chunks > 1 (requests
 // of at most 64 packed rows): the key tiles in that many shares over blocks, and a merge.
 CB_EXPORT int cb_attention_mma_sink(const void* q, int q_stride, void* out, int out_stride,
                                     const void* gate, int gate_stride, const void* k_cache,
                                     const void* v_cache, const float* sinks, const int* req_row_start,
                                     const int* req_first_pos, const int* block_table, int table_stride,
                                     int n_requests, int max_new_tokens, int n_heads, int n_kv_heads,
-                                    int head_dim, int page_tokens, float scale, int window,
-                                    int keep_first, float out_scale, float* partial, int n_chunks,
+                                    int head_dim, int value_dim, int page_tokens, float scale, int window,
+                                    int chunked, int keep_first, float out_scale, float* partial, int n_chunks,
                                     int gate_per_head, void* stream) {
     if (n_requests <= 0 || max_new_tokens <= 0) return 0;
-    if (head_dim <= 0 || head_dim > 256 || (head_dim & 15) || n_heads % n_kv_heads != 0 ||
-        (q_stride & 7) || (out_stride & 1) || (!gate_per_head && (gate_stride & 1)) || ((uintptr_t)q & 15) ||
+    if (head_dim <= 0 || head_dim > 256 || (head_dim & 15) || value_dim <= 0 || value_dim > 256 ||
+        (value_dim & 15) || n_heads % n_kv_heads != 0 || (q_stride & 7) || (out_stride & 1) || (!gate_per_head && (gate_stride & 1)) || ((uintptr_t)q & 15) ||
         ((uintptr_t)out & 3) || (!gate_per_head && ((uintptr_t)gate & 3)) || ((uintptr_t)k_cache & 15) ||
         ((uintptr_t)v_cache & 15) || keep_first < 0)
         return CB_ERR_UNSUPPORTED;
@@ -1076,27 +1135,30 @@ CB_EXPORT int cb_attention_mma_sink(const void* q, int q_stride, void* out, int 
     p.gate_stride = gate_stride;
     p.gate_per_head = gate != nullptr && gate_per_head ? 1 : 0;
     p.out_scale = out_scale;
+    p.value_dim = value_dim;
+    p.chunked = window > 0 && chunked ? 1 : 0;
     p.partial = partial;
     p.n_chunks = n_chunks;
     p.chunk_keys = SPLIT_KEYS;
     cudaStream_t s = (cudaStream_t)stream;
     const int max_rows = max_new_tokens * (n_heads / n_kv_heads);
+    const int wide = head_dim > value_dim ? head_dim : value_dim;
     if (n_chunks > 1) {
         // the key tiles of every request's (single) row tile in n_chunks shares, then a merge;
-        // partial: n_requests * n_kv_heads * n_chunks * max_rows * (head_dim + 2) floats
+        // partial: n_requests * n_kv_heads * n_chunks * max_rows * (value_dim + 2) floats
         if (partial == nullptr || max_rows > 64 || n_chunks > 32) return CB_ERR_UNSUPPORTED;
         p.chunk_keys = max_rows;
-        if (head_dim <= 16) return launch_tiles_split<16>(p, n_requests, max_rows, s);
-        if (head_dim <= 32) return launch_tiles_split<32>(p, n_requests, max_rows, s);
-        if (head_dim <= 64) return launch_tiles_split<64>(p, n_requests, max_rows, s);
-        if (head_dim <= 128) return launch_tiles_split<128>(p, n_requests, max_rows, s);
+        if (wide <= 16) return launch_tiles_split<16>(p, n_requests, max_rows, s);
+        if (wide <= 32) return launch_tiles_split<32>(p, n_requests, max_rows, s);
+        if (wide <= 64) return launch_tiles_split<64>(p, n_requests, max_rows, s);
+        if (wide <= 128) return launch_tiles_split<128>(p, n_requests, max_rows, s);
         return launch_tiles_split<256>(p, n_requests, max_rows, s);
     }
     p.n_chunks = 0;
     const int q_tiles = (max_rows + 63) / 64;
-    if (head_dim <= 16) return launch_tiles<16, true>(p, n_requests, q_tiles, s);
-    if (head_dim <= 32) return launch_tiles<32, true>(p, n_requests, q_tiles, s);
-    if (head_dim <= 64) return launch_tiles<64, true>(p, n_requests, q_tiles, s);
-    if (head_dim <= 128) return launch_tiles<128, true>(p, n_requests, q_tiles, s);
+    if (wide <= 16) return launch_tiles<16, true>(p, n_requests, q_tiles, s);
+    if (wide <= 32) return launch_tiles<32, true>(p, n_requests, q_tiles, s);
+    if (wide <= 64) return launch_tiles<64, true>(p, n_requests, q_tiles, s);
+    if (wide <= 128) return launch_tiles<128, true>(p, n_requests, q_tiles, s);
     return launch_tiles<256, true>(p, n_requests, q_tiles, s);
 }

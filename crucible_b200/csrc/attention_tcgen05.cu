@@ -58,6 +58,10 @@ struct TcAttnParams {
     float scale_log2;
     int window;
     int keep_first;          // with a window: keys before this position stay visible to every later row
+    int chunked;             // 1: `window` is the size of chunks counted from position 0: a row reads
+                             // the keys of its own chunk up to itself
+    float out_scale;         // every result times this
+    const float* sinks;      // [n_heads] or null: exp(sink) joins a row's denominator, with no value
     int n_pages;             // of the pool
     int runs;                // 1: the 4-D maps may be used for tiles whose pages are consecutive
     int* status;
@@ -104,6 +108,12 @@ struct Storage {
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
+}
+
+// The first key that a row at position `pos` reads behind the kept first tokens.
+__device__ __forceinline__ int first_key(const TcAttnParams& p, int pos) {
+    if (p.window <= 0) return 0;
+    return p.chunked ? pos - pos % p.window : max(0, pos - p.window + 1);
 }
 
 // 2^x by the special-function unit, flushing denormals: the argument is a score
@@ -199,7 +209,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
     const int last_row = min(n_rows - 1, qt * ROWS + ROWS - 1);
     const int max_pos = first_pos + last_row / n_rep;
     const int min_pos = first_pos + (qt * ROWS) / n_rep;
-    int key_lo = p.window > 0 ? max(0, min_pos - p.window + 1) : 0;
+    int key_lo = first_key(p, min_pos);
     key_lo = key_lo / KEYS * KEYS;
     const int key_end = max_pos + 1;
     // kept first tokens: their tiles that lie wholly before the window's first tile come first
@@ -457,7 +467,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
         // rows past the request's last are computed like rows that may read every key (their
         // queries are zero) and are not stored: they keep a tile's fast path open
         const int pos = real ? first_pos + row / n_rep : (1 << 30);
-        const int lo = real && p.window > 0 ? max(0, pos - p.window + 1) : 0;
+        const int lo = real ? first_key(p, pos) : 0;
         const uint32_t lane_bits = (uint32_t)(quarter * 32) << 16;
         float m_ref = -INFINITY, l = 0.f;
         bool ok = true;
@@ -581,8 +591,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
         const int j_last = group + (my_tiles - 1) * GROUPS;
         if (ok && my_tiles > 0) ok = wait_all(&s.pv_done[j_last % PB], (j_last / PB) & 1);
         __nv_bfloat16* dst = nullptr;
+        float sink = -INFINITY;                       // in the base-2 exponent
         if (real) {
             const int tok = row_base + row / n_rep, head = kv_head * n_rep + row % n_rep;
+            if (p.sinks != nullptr) sink = p.sinks[head] * LOG2E;
             dst = p.out + (size_t)tok * p.out_stride + (size_t)head * HD;
         }
         if (GROUPS > 1) {
@@ -595,11 +607,12 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                 tc::tc_fence_after_sync();
                 const float2 other = s.merge[group ^ 1][r];
                 const float m_mine = my_tiles > 0 ? m_ref : -INFINITY;
-                const float m_all = fmaxf(m_mine, other.x);
+                const float m_all = fmaxf(fmaxf(m_mine, other.x), sink);
                 const float f_mine = m_mine == -INFINITY ? 0.f : exp2f(m_mine - m_all);
                 const float f_other = other.x == -INFINITY ? 0.f : exp2f(other.x - m_all);
-                const float l_all = (my_tiles > 0 ? l : 0.f) * f_mine + other.y * f_other;
-                const float inv = l_all > 0.f ? 1.0f / l_all : 0.f;
+                float l_all = (my_tiles > 0 ? l : 0.f) * f_mine + other.y * f_other;
+                if (sink != -INFINITY) l_all += exp2f(sink - m_all);
+                const float inv = l_all > 0.f ? p.out_scale / l_all : 0.f;
                 const float w_mine = f_mine * inv, w_other = f_other * inv;
                 const int c0 = group * 32;
                 uint32_t a[32], b[32];
@@ -630,7 +643,12 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
             }
         } else if (ok && n_tiles > 0) {
             tc::tc_fence_after_sync();
-            const float inv = l > 0.f ? 1.0f / l : 0.f;
+            float inv = l > 0.f ? p.out_scale / l : 0.f;
+            if (sink != -INFINITY) {
+                const float top = fmaxf(m_ref, sink);
+                const float keep = exp2f(m_ref - top);
+                inv = keep * p.out_scale / (l * keep + exp2f(sink - top));
+            }
 #pragma unroll 1
             for (int c0 = 0; c0 < HD; c0 += 32) {
                 uint32_t v[32];
@@ -679,13 +697,14 @@ int launch_as(dim3 grid, cudaStream_t st, const CUtensorMap& mk, const CUtensorM
 // Attention for the rows of a step whose requests bring portions of prompts.
 // k_cache / v_cache: [n_pages][n_kv_heads][page_tokens][head_dim] bf16; head_dim 64 or 128.
 // keep_first (with a window): a row at position p reads j <= p with p - j < window or j < keep_first.
+// chunked: `window` is a chunk's size (first_key).  sinks: [n_heads] or null.  Results times out_scale.
 CB_EXPORT int cb_attention_tcgen05_kept(const void* qkv, int qkv_stride, void* out, int out_stride,
                                         const void* k_cache, const void* v_cache, int n_pages,
                                         const int* req_row_start, const int* req_first_pos,
                                         const int* block_table, int table_stride, int n_requests,
                                         int max_new_tokens, int n_heads, int n_kv_heads, int head_dim,
-                                        int page_tokens, float scale, int window, int keep_first, int lean,
-                                        int* status, void* stream) {
+                                        int page_tokens, float scale, int window, int chunked, int keep_first,
+                                        float out_scale, const float* sinks, int lean, int* status, void* stream) {
     if (n_requests <= 0 || max_new_tokens <= 0) return 0;
     if (keep_first < 0 || !(scale > 0.f)) return CB_ERR_UNSUPPORTED;
     if ((head_dim != 64 && head_dim != 128) || n_heads % n_kv_heads != 0 || page_tokens < 8 || page_tokens > KEYS ||
@@ -725,6 +744,9 @@ CB_EXPORT int cb_attention_tcgen05_kept(const void* qkv, int qkv_stride, void* o
     p.scale_log2 = scale * LOG2E;
     p.window = window;
     p.keep_first = window > 0 ? keep_first : 0;
+    p.chunked = window > 0 && chunked ? 1 : 0;
+    p.sinks = sinks;
+    p.out_scale = out_scale;
     p.status = status;
     const int n_rep = n_heads / n_kv_heads;
     const int q_tiles = (max_new_tokens * n_rep + ROWS - 1) / ROWS;
@@ -751,5 +773,5 @@ CB_EXPORT int cb_attention_tcgen05(const void* qkv, int qkv_stride, void* out, i
                                    void* stream) {
     return cb_attention_tcgen05_kept(qkv, qkv_stride, out, out_stride, k_cache, v_cache, n_pages, req_row_start,
                                      req_first_pos, block_table, table_stride, n_requests, max_new_tokens, n_heads,
-                                     n_kv_heads, head_dim, page_tokens, scale, window, 0, lean, status, stream);
+                                     n_kv_heads, head_dim, page_tokens, scale, window, 0, 0, 1.0f, nullptr, lean, status, stream);
 }

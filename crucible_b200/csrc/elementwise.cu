@@ -273,6 +273,26 @@ CB_EXPORT int cb_add_vector(float* x, const float* v, int n_rows, int width, voi
     return cb_last_error();
 }
 
+// x[t] += rows[t], then += v (may be null)
+__global__ void add_rows_kernel(float* __restrict__ x, const float* __restrict__ rows,
+                                const float* __restrict__ v, int width) {
+    cb_pdl_trigger();
+    cb_pdl_wait();
+    float* row = x + (size_t)blockIdx.x * width;
+    const float* add = rows + (size_t)blockIdx.x * width;
+    for (int i = threadIdx.x; i < width; i += blockDim.x) {
+        const float s = row[i] + add[i];
+        row[i] = v != nullptr ? s + v[i] : s;
+    }
+}
+
+CB_EXPORT int cb_add_rows(float* x, const float* rows, const float* v, int n_rows, int width, void* stream) {
+    if (n_rows <= 0) return 0;
+    cb_launch(add_rows_kernel, dim3(n_rows), dim3(width >= 1024 ? 256 : 128), 0, (cudaStream_t)stream, x, rows, v,
+              width);
+    return cb_last_error();
+}
+
 __global__ void softcap_kernel(float* __restrict__ z, int width, float cap, float inv_cap) {
     cb_pdl_trigger();
     cb_pdl_wait();

@@ -5,14 +5,19 @@
 //
 // Everything is decided on the device, so a step's launches depend on its shape only:
 //   route    one warp per token: the top logits, their softmax, and each (token, choice)
-//            pair's place among its expert's pairs (a counter per expert)
+//            pair's place among its expert's pairs (a counter per expert); the experts may form
+//            equal groups of neighbours of which only the best few take part (a group's score is
+//            its best logit), and slices of a shared expert may ride along as experts that every
+//            token chooses, weighted by the sigmoid of one logit of the token
 //   plan     one block: where each expert's pairs start in the sorted order, the list of
 //            row tiles (an expert, a start, a count), and the sorted order itself
 //   tiles    gate/up with the gated pair (SiLU, or the capped form), then down times the pair's weight: a block owns a tile of
 //            rows of one expert and a tile of columns; rows beyond the tile's count and
 //            tiles beyond the plan's count do nothing.  fp32 sums over ascending k, so a
 //            pair's result does not depend on which other pairs share its tile.
-//   combine  residual[t] += the token's pairs in the order of its choices.
+//   combine  residual[t] += the token's pairs in the order of its choices (or, for the tensor
+//            cores' grouped products, the token's rows of the sorted order times their weights),
+//            and a shared expert's row times the token's gate if it was run apart.
 #define CB_PDL_BIT 13      // this file's bit in CRUCIBLE_PDL
 #include "common.cuh"
 
@@ -32,9 +37,10 @@ __device__ __forceinline__ float gated_f(float g, float u, const GateRule& p) {
 }
 
 __global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
-                                 int n_tokens, int E, int top,
+                                 int n_tokens, int stride, int E, int top,
                                  int* __restrict__ idx, float* __restrict__ weight,
-                                 int* __restrict__ place, int* __restrict__ count) {
+                                 int* __restrict__ place, int* __restrict__ count, int groups, int keep,
+                                 int n_shared, int gate_col, float scale, float* __restrict__ gate_out) {
     cb_pdl_trigger();
     cb_pdl_wait();
     const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -44,7 +50,33 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
 #pragma unroll
     for (int i = 0; i < MAX_PER_LANE; ++i) {
         const int e = lane + 32 * i;
-        v[i] = e < E ? logits[(size_t)t * E + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
+        v[i] = e < E ? logits[(size_t)t * stride + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
+    }
+    if (keep < groups) {
+        // only the experts of the `keep` groups with the largest best logit (the lower group on
+        // equal ones) stay
+        __shared__ float all[4][32 * MAX_PER_LANE], best_of[4][32 * MAX_PER_LANE];
+        const int warp = threadIdx.x >> 5, size = E / groups;
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i)
+            if (lane + 32 * i < E) all[warp][lane + 32 * i] = v[i];
+        __syncwarp();
+        for (int g = lane; g < groups; g += 32) {
+            float m = -INFINITY;
+            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, all[warp][e]);
+            best_of[warp][g] = m;
+        }
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < MAX_PER_LANE; ++i) {
+            const int e = lane + 32 * i;
+            if (e >= E) continue;
+            const int mine_g = e / size;
+            const float m = best_of[warp][mine_g];
+            int ahead = 0;
+            for (int g = 0; g < groups; ++g) ahead += best_of[warp][g] > m || (best_of[warp][g] == m && g < mine_g);
+            if (ahead >= keep) v[i] = -INFINITY;
+        }
     }
     float first = 0.f, total = 0.f, mine = 0.f;
     int mine_e = 0;
@@ -71,10 +103,22 @@ __global__ void moe_route_kernel(const float* __restrict__ logits, const float* 
         total += p;
         if (lane == j) { mine = p; mine_e = best_e; }
     }
+    const size_t at = (size_t)t * (top + n_shared);
     if (lane < top) {
-        idx[(size_t)t * top + lane] = mine_e;
-        weight[(size_t)t * top + lane] = mine / total;
-        place[(size_t)t * top + lane] = atomicAdd(&count[mine_e], 1);
+        idx[at + lane] = mine_e;
+        weight[at + lane] = mine / total * scale;
+        place[at + lane] = atomicAdd(&count[mine_e], 1);
+    }
+    if (gate_col >= 0) {
+        const float gate = scale / (1.0f + expf(-logits[(size_t)t * stride + gate_col]));
+        // the shared expert's slices: every token's, so its place among their pairs is its own number
+        for (int s = lane; s < n_shared; s += 32) {
+            idx[at + top + s] = E + s;
+            weight[at + top + s] = gate;
+            place[at + top + s] = t;
+            if (t == 0) count[E + s] = n_tokens;
+        }
+        if (gate_out != nullptr && lane == 0) gate_out[t] = gate;
     }
 }
 
@@ -301,15 +345,39 @@ __global__ void __launch_bounds__(256, 3) moe_rows_small_kernel(
     }
 }
 
-__global__ void moe_combine_kernel(const float* __restrict__ pair_out, int top, float* __restrict__ residual,
-                                   int width) {
+// rows: by pair, weighted already (offsets null), or in the sorted order, where a pair's row lies at
+// its expert's start + its place and takes its weight here.  shared (may be null): rows by token,
+// times gate[token].  V: vector width.
+template <int V>
+__global__ void moe_combine_kernel(const float* __restrict__ rows, int top, float* __restrict__ residual,
+                                   int width, const int* __restrict__ offsets, const int* __restrict__ idx,
+                                   const int* __restrict__ place, const float* __restrict__ weight,
+                                   const float* __restrict__ shared, const float* __restrict__ gate) {
     cb_pdl_trigger();
     cb_pdl_wait();
     const int t = blockIdx.x;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-        float sum = 0.f;
-        for (int j = 0; j < top; ++j) sum += pair_out[((size_t)t * top + j) * width + i];
-        residual[(size_t)t * width + i] += sum;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+        float sum[V];
+#pragma unroll
+        for (int e = 0; e < V; ++e) sum[e] = 0.f;
+        auto add = [&](const float* src, float w) {
+            if constexpr (V == 4) {
+                const float4 a = *reinterpret_cast<const float4*>(src);
+                sum[0] = fmaf(w, a.x, sum[0]); sum[1] = fmaf(w, a.y, sum[1]);
+                sum[2] = fmaf(w, a.z, sum[2]); sum[3] = fmaf(w, a.w, sum[3]);
+            } else {
+                sum[0] = fmaf(w, src[0], sum[0]);
+            }
+        };
+        for (int j = 0; j < top; ++j) {
+            const size_t p = (size_t)t * top + j;
+            if (offsets == nullptr) add(rows + p * width + i, 1.0f);
+            else add(rows + (size_t)(offsets[idx[p]] + place[p]) * width + i, weight[p]);
+        }
+        if (shared != nullptr) add(shared + (size_t)t * width + i, gate[t]);
+        float* dst = residual + (size_t)t * width + i;
+#pragma unroll
+        for (int e = 0; e < V; ++e) dst[e] += sum[e];
     }
 }
 
@@ -324,32 +392,30 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, int h_stride, const i
     for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = src[i];
 }
 
-// pair_out[pair] = weight[pair] * rows[sorted place of the pair]
-__global__ void moe_scatter_kernel(const float* __restrict__ rows, const int* __restrict__ sorted_pair,
-                                   const float* __restrict__ weight, float* __restrict__ pair_out, int width) {
-    cb_pdl_trigger();
-    cb_pdl_wait();
-    const int p = sorted_pair[blockIdx.x];
-    const float wt = weight[p];
-    for (int i = threadIdx.x; i < width; i += blockDim.x)
-        pair_out[(size_t)p * width + i] = wt * rows[(size_t)blockIdx.x * width + i];
-}
-
 }  // namespace
 
 CB_EXPORT int cb_moe_tile_rows() { return TM; }
 
-CB_EXPORT int cb_moe_route(const float* logits, const float* bias, int n_tokens, int E, int top, int* idx,
-                           float* weight,
+// logits: rows at `stride`, the first E of them the experts'.  groups, keep: equal groups of
+// neighbouring experts of which `keep` take part (groups == keep: no restriction).  gate_col >= 0: the
+// column of the shared expert's gate logit; n_shared slices of it ride along as experts E .. E +
+// n_shared - 1 of every token, and gate_out (may be null) receives scale * sigmoid of that logit.
+// scale: on every weight.  count and plan cover E + n_shared experts, a token has top + n_shared pairs.
+CB_EXPORT int cb_moe_route(const float* logits, int stride, const float* bias, int n_tokens, int E, int top,
+                           int* idx, float* weight,
                            int* place, int* count, int* plan, int max_tiles, int* sorted_pair,
-                           int tile_rows, void* stream) {
+                           int tile_rows, int groups, int keep, int n_shared, int gate_col, float scale,
+                           float* gate_out, void* stream) {
     if (n_tokens <= 0) return 0;
     if (E > 32 * MAX_PER_LANE || top > E || top <= 0 || top > 32) return CB_ERR_UNSUPPORTED;
+    if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups) || n_shared < 0 ||
+        (n_shared > 0 && gate_col < 0) || gate_col >= stride)
+        return CB_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    cb_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, s, logits, bias, n_tokens, E, top, idx,
-              weight, place, count);
-    cb_launch(moe_plan_kernel, dim3(1), dim3(256), 0, s, count, E, n_tokens * top, (const int*)idx,
-              (const int*)place, plan, max_tiles, sorted_pair, tile_rows > 0 ? tile_rows : TM);
+    cb_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, s, logits, bias, n_tokens, stride, E, top,
+              idx, weight, place, count, groups, keep, n_shared, gate_col, scale, gate_out);
+    cb_launch(moe_plan_kernel, dim3(1), dim3(256), 0, s, count, E + n_shared, n_tokens * (top + n_shared),
+              (const int*)idx, (const int*)place, plan, max_tiles, sorted_pair, tile_rows > 0 ? tile_rows : TM);
     return cb_last_error();
 }
 
@@ -408,11 +474,23 @@ CB_EXPORT int cb_moe_rows_small(int gated, const void* a, int a_stride, const vo
     return cb_last_error();
 }
 
-CB_EXPORT int cb_moe_combine(const float* pair_out, int top, float* residual, int n_tokens, int width,
-                             void* stream) {
+// plan null: rows [tokens * top][width] by pair, weighted; else rows in the sorted order of that plan.
+// shared (or null): rows [tokens][width] that join with gate[token].
+CB_EXPORT int cb_moe_combine(const float* rows, int top, float* residual, int n_tokens, int width,
+                             const int* plan, const int* idx, const int* place, const float* weight,
+                             const float* shared, const float* gate, void* stream) {
     if (n_tokens <= 0) return 0;
-    cb_launch(moe_combine_kernel, dim3(n_tokens), dim3(width >= 1024 ? 256 : 128), 0, (cudaStream_t)stream,
-              pair_out, top, residual, width);
+    const int* offsets = plan != nullptr ? plan + 1 : nullptr;
+    const bool vec = (width & 3) == 0 && ((uintptr_t)rows & 15) == 0 && ((uintptr_t)residual & 15) == 0 &&
+                     ((uintptr_t)shared & 15) == 0;
+    const dim3 block(width >= 1024 ? 256 : 128);
+    cudaStream_t s = (cudaStream_t)stream;
+    if (vec)
+        cb_launch(moe_combine_kernel<4>, dim3(n_tokens), block, 0, s, rows, top, residual, width, offsets, idx, place,
+                  weight, shared, gate);
+    else
+        cb_launch(moe_combine_kernel<1>, dim3(n_tokens), block, 0, s, rows, top, residual, width, offsets, idx, place,
+                  weight, shared, gate);
     return cb_last_error();
 }
 
@@ -426,13 +504,5 @@ CB_EXPORT int cb_moe_gather(const void* h, int h_stride, int dtype, const int* s
     else
         cb_launch(moe_gather_kernel<__nv_bfloat16>, dim3(n_pairs), dim3(128), 0, s, (const __nv_bfloat16*)h,
                   h_stride, sorted_pair, top, (__nv_bfloat16*)out, width);
-    return cb_last_error();
-}
-
-CB_EXPORT int cb_moe_scatter(const float* rows, const int* sorted_pair, const float* weight,
-                             float* pair_out, int n_pairs, int width, void* stream) {
-    if (n_pairs <= 0) return 0;
-    cb_launch(moe_scatter_kernel, dim3(n_pairs), dim3(128), 0, (cudaStream_t)stream, rows, sorted_pair,
-              weight, pair_out, width);
     return cb_last_error();
 }

@@ -1,12 +1,15 @@
 // Mixers that carry a matrix of fixed size per head from token to token instead of
 // a cache of keys: the gated delta rule, the matrix memory with exponential gates
 // (mLSTM), the wkv rule with a decay per key channel and a bonus for the current token,
-// and the state-space rule with one decay per head (Mamba-2).  Per request and head the state is S [D][E] in fp32 (mLSTM also n [D] and
+// the state-space rule with one decay per head (Mamba-2), and the delta rule with a decay per
+// key channel.  Per request and head the state is S [D][E] in fp32 (mLSTM also n [D] and
 // a running maximum m); it lives in the request's state slot and is read at the
 // start of a step and written at its end, so a prompt may be cut anywhere.
 //
 //   delta rule, per token:  S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 //                           (the kernel takes both dots from S before the write: see there)
+//   channel delta, per token:  S <- diag(g) S, the rest like the delta rule (g a vector over the
+//                           key channels of the head)
 //   mLSTM, per token:       m' = max(f + m, i);  a = exp(f + m - m');  b = exp(i - m');
 //                           S <- a S + b k v^T;  n <- a n + b k;
 //                           o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
@@ -33,7 +36,9 @@
 
 namespace {
 
-constexpr int RULE_DELTA = 0, RULE_MLSTM = 1, RULE_WKV = 2, RULE_SSD = 3;
+constexpr int RULE_DELTA = 0, RULE_MLSTM = 1, RULE_WKV = 2, RULE_SSD = 3, RULE_CHANNEL = 4;
+// rules whose decay is a vector of D per token and head, staged beside k and q
+template <int RULE> constexpr bool VECTOR_DECAY = RULE == RULE_WKV || RULE == RULE_CHANNEL;
 constexpr int GATE_SILU = 0, GATE_SIGMOID = 1;
 constexpr int THREADS = 128;      // of a recurrence block: 128 / LANES columns of S
 constexpr int CHUNK = 16;         // tokens staged at a time
@@ -134,6 +139,138 @@ __global__ void conv_tail_update_kernel(const T* __restrict__ proj, int proj_str
     }
 }
 
+// ---- channel delta: convolution + SiLU, unit q and k, decays per key channel, beta ----------
+// proj row: [q: G*D | k: G*D | v: H*E | ...] in T, C = 2*G*D + H*E channels under the convolution;
+// conv_w: fp32 [taps][C], the last row meets the current token; the request's state holds the last
+// taps - 1 inputs of every channel, oldest first, fp32 [taps-1][C].  rate: fp32 rows of H*D logits,
+// beta_logit: fp32 rows of H.  Writes qkv fp32 [rows][C + H*D] = [q | k | v | decay], decay =
+// exp(-exp(A_log_h) softplus(rate + dt_bias)), and beta fp32 [rows][H].
+// One warp takes a tile of a request's tokens (grid y: tiles, z: requests) and one unit: a q or k
+// head, 128 channels of v, 128 channels of the decays, or the betas; it walks the tokens down its
+// channels with the last inputs in registers.  The first tile's warp alone reads the old state and
+// then writes the new one for its own channels.
+constexpr int CHANNEL_TILE = 8, CHANNEL_RUN = 128;
+
+template <typename T, int NV, int TAPS>
+__device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, int proj_stride,
+                                                  const float* __restrict__ conv_w, int taps_, int C, int c0,
+                                                  int count, bool unit, float unit_scale, float* tail,
+                                                  int row0, int n, int a, int b, bool first,
+                                                  float* __restrict__ qkv, int width) {
+    const int taps = TAPS > 0 ? TAPS : taps_, keep = taps - 1;
+    const int lane = threadIdx.x & 31;
+    constexpr int W = TAPS > 0 ? TAPS : 1;
+    float past[NV][W], wt[NV][W];
+    // the input of channel c0 + lane + 32 i at the portion's token `row` (negative: from the state)
+    auto input = [&](int row, int c) {
+        return row >= 0 ? cb_to_float(proj[(size_t)(row0 + row) * proj_stride + c])
+                        : tail[(size_t)(keep + row) * C + c];
+    };
+    if (TAPS > 0) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = c0 + lane + 32 * i;
+            const bool in = lane + 32 * i < count;
+#pragma unroll
+            for (int j = 0; j < W; ++j) {
+                wt[i][j] = in ? conv_w[(size_t)j * C + c] : 0.f;
+                past[i][j] = (in && j < W - 1) ? input(a - (W - 1) + j, c) : 0.f;
+            }
+        }
+    }
+    for (int t = a; t < b; ++t) {
+        float v[NV];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = c0 + lane + 32 * i;
+            const bool in = lane + 32 * i < count;
+            float acc = 0.f;
+            if (TAPS > 0) {
+                past[i][W - 1] = in ? input(t, c) : 0.f;
+#pragma unroll
+                for (int j = 0; j < W; ++j) acc = fmaf(wt[i][j], past[i][j], acc);
+#pragma unroll
+                for (int j = 0; j < W - 1; ++j) past[i][j] = past[i][j + 1];
+            } else if (in) {
+                for (int j = 0; j < taps; ++j) acc = fmaf(conv_w[(size_t)j * C + c], input(t - keep + j, c), acc);
+            }
+            v[i] = in ? silu_f(acc) : 0.f;
+            ss = fmaf(v[i], v[i], ss);
+        }
+        float inv = 1.0f;
+        if (unit) inv = unit_scale / sqrtf(cb_warp_sum(ss) + 1e-6f);
+        float* dst = qkv + (size_t)(row0 + t) * width + c0;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (lane + 32 * i < count) dst[lane + 32 * i] = unit ? v[i] * inv : v[i];
+    }
+    if (first) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int c = c0 + lane + 32 * i;
+            if (lane + 32 * i >= count) continue;
+            for (int k = 0; k < keep; ++k)          // ascending: reads run ahead of writes
+                tail[(size_t)k * C + c] = input(n - keep + k, c);
+        }
+    }
+}
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(128) channel_delta_prepare_kernel(
+    const T* __restrict__ proj, int proj_stride, const float* __restrict__ conv_w, int taps,
+    const float* __restrict__ rate, int rate_stride, const float* __restrict__ beta_logit, int beta_stride,
+    const float* __restrict__ a_log, const float* __restrict__ dt_bias, const int* __restrict__ req_row_start,
+    const int* __restrict__ req_state_slot, unsigned char* state, long slot_stride, long tail_off,
+    float* __restrict__ qkv, float* __restrict__ beta, int H, int G, int D, int E, int n_units, int tile) {
+    cb_pdl_trigger();
+    cb_pdl_wait();
+    int unit = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (unit >= n_units) return;
+    const int lane = threadIdx.x & 31;
+    const int req = blockIdx.z;
+    const int row0 = req_row_start[req], n = req_row_start[req + 1] - row0;
+    const int a = blockIdx.y * tile, b = min(n, a + tile);
+    if (a >= n) return;
+    const int C = 2 * G * D + H * E, width = C + H * D;
+    float* tail = state_at(state, slot_stride, req_state_slot[req], tail_off);
+    const bool first = blockIdx.y == 0;
+    if (unit < 2 * G) {
+        const float sc = unit < G ? 1.0f / sqrtf((float)D) : 1.0f;
+        if (D <= 128)
+            channel_conv_unit<T, 4, TAPS>(proj, proj_stride, conv_w, taps, C, unit * D, D, true, sc, tail, row0, n,
+                                          a, b, first, qkv, width);
+        else
+            channel_conv_unit<T, 8, TAPS>(proj, proj_stride, conv_w, taps, C, unit * D, D, true, sc, tail, row0, n,
+                                          a, b, first, qkv, width);
+        return;
+    }
+    unit -= 2 * G;
+    const int v_runs = (H * E + CHANNEL_RUN - 1) / CHANNEL_RUN;
+    if (unit < v_runs) {
+        const int at = unit * CHANNEL_RUN;
+        channel_conv_unit<T, 4, TAPS>(proj, proj_stride, conv_w, taps, C, 2 * G * D + at, min(CHANNEL_RUN, H * E - at),
+                                      false, 1.0f, tail, row0, n, a, b, first, qkv, width);
+        return;
+    }
+    unit -= v_runs;
+    const int d_runs = (H * D + CHANNEL_RUN - 1) / CHANNEL_RUN;
+    if (unit < d_runs) {
+        const int at = unit * CHANNEL_RUN;
+        for (int i = lane; i < min(CHANNEL_RUN, H * D - at); i += 32) {
+            const float speed = -expf(a_log[(at + i) / D]), bias = dt_bias[at + i];
+            for (int t = a; t < b; ++t)
+                qkv[(size_t)(row0 + t) * width + C + at + i] =
+                    expf(speed * softplus_f(rate[(size_t)(row0 + t) * rate_stride + at + i] + bias));
+        }
+        return;
+    }
+    for (int i = lane; i < (b - a) * H; i += 32) {
+        const int t = row0 + a + i / H, h = i % H;
+        beta[(size_t)t * H + h] = sigmoid_f(beta_logit[(size_t)t * beta_stride + h]);
+    }
+}
+
 // ---- mLSTM: q * D^-1/2, k, v to fp32 and the capped log gates -----------------------------
 // proj row: [q: H*D | k: H*D | v: H*E | ...]; gates: fp32 [rows][2H] = [input | forget] logits.
 template <typename T>
@@ -224,14 +361,15 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
     unsigned char* state, long slot_stride, long s_off, long n_off, long m_off,
     float* __restrict__ out, int n_heads, int n_qk_heads, int D, int E, int w_off,
     const float* __restrict__ per_head) {
-    // w_off: wkv's decay vectors in the rows of qkv (one of D per head); per_head: wkv's bonus
+    // w_off: wkv's and channel delta's decay vectors in the rows of qkv (one of D per head); per_head: wkv's bonus
     // u [H][D], the state-space rule's skip [H]
     cb_pdl_trigger();
     cb_pdl_wait();
     constexpr int COLS = THREADS / LANES;
     constexpr int PAD = P == 4 ? 8 : 4;       // the parts' 16-byte reads then fall on different banks
     constexpr int PITCH = LANES * (P + PAD);
-    constexpr int NVEC = RULE == RULE_WKV ? 3 : 2;      // staged vectors of D per token: k, q (, w)
+    constexpr bool VECTOR = VECTOR_DECAY<RULE>;
+    constexpr int NVEC = VECTOR ? 3 : 2;      // staged vectors of D per token: k, q (, w)
     constexpr int BUF = CHUNK * (NVEC * PITCH + COLS) + 2 * CHUNK;      // floats of one stage
     extern __shared__ __align__(16) float stage[];
     const int r = blockIdx.x, head = blockIdx.y, col0 = blockIdx.z * COLS;
@@ -259,14 +397,14 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
     if (RULE == RULE_MLSTM) m = *M;
     __syncthreads();
     // 16-byte copies if every row of q and k starts on a 16-byte boundary
-    const bool vec = ((C | q_off | k_off | D | (RULE == RULE_WKV ? w_off : 0)) & 3) == 0;
+    const bool vec = ((C | q_off | k_off | D | (VECTOR ? w_off : 0)) & 3) == 0;
     // a chunk's q, k, v and gates on their way into one of the two stages (asynchronous
     // copies: the next chunk travels while this one is worked on)
     auto fetch = [&](int base, int buf) {
         float* sk = stage + buf * BUF;
         float* sq = sk + CHUNK * PITCH;
         float* sv = sq + (NVEC - 1) * CHUNK * PITCH;
-        float* sw = sq + CHUNK * PITCH;                     // wkv only
+        float* sw = sq + CHUNK * PITCH;                     // rules with a vector of decays only
         float* s0 = sv + CHUNK * COLS;
         float* s1 = s0 + CHUNK;
         const int cnt = min(CHUNK, row1 - base);
@@ -278,7 +416,7 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
                 const int at = tt * PITCH + d + (d / P) * PAD;
                 cp_async<16>(sk + at, src + k_off);
                 cp_async<16>(sq + at, src + q_off);
-                if (RULE == RULE_WKV) cp_async<16>(sw + at, src + w_off);
+                if (VECTOR) cp_async<16>(sw + at, src + w_off + (size_t)(head - g) * D);
             }
         } else {
             for (int i = threadIdx.x; i < cnt * D; i += blockDim.x) {
@@ -287,7 +425,7 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
                 const int at = tt * PITCH + d + (d / P) * PAD;
                 cp_async<4>(sk + at, src + k_off);
                 cp_async<4>(sq + at, src + q_off);
-                if (RULE == RULE_WKV) cp_async<4>(sw + at, src + w_off);
+                if (VECTOR) cp_async<4>(sw + at, src + w_off + (size_t)(head - g) * D);
             }
         }
         for (int i = threadIdx.x; i < cnt * COLS; i += blockDim.x) {
@@ -296,7 +434,8 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
                 cp_async<4>(sv + i, qkv + (size_t)(base + tt) * C + v_off + (size_t)head * E + col0 + c);
         }
         if (RULE != RULE_WKV && threadIdx.x < cnt) {
-            cp_async<4>(s0 + threadIdx.x, sc0 + (size_t)(base + threadIdx.x) * n_heads + head);
+            if (RULE != RULE_CHANNEL)
+                cp_async<4>(s0 + threadIdx.x, sc0 + (size_t)(base + threadIdx.x) * n_heads + head);
             cp_async<4>(s1 + threadIdx.x, sc1 + (size_t)(base + threadIdx.x) * n_heads + head);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
@@ -366,6 +505,40 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
 #pragma unroll
                 for (int i = 0; i < P; ++i) k_prev[i] = kk[i];
                 g_prev = decay;
+                u_prev = u;
+            } else if (RULE == RULE_CHANNEL) {
+                // As the delta rule: the write of the token before is applied on the way, then this
+                // token's decays; with r = S^T k and w = S^T q over what that leaves:
+                //   u = beta (v - r),   o = w + u (k . q)       [= (S + k u^T)^T q]
+                const float beta = s1[tt];
+                const float4* w4 = reinterpret_cast<const float4*>(sw + tt * PITCH + part * (P + PAD));
+                float rk[4] = {0.f, 0.f, 0.f, 0.f}, rq[4] = {0.f, 0.f, 0.f, 0.f}, kq[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+                for (int j = 0; j < P / 4; ++j) {
+                    const float4 a = w4[j];
+                    const float ww[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        const int i = 4 * j + e;
+                        s[i] = __fmul_rn(ww[e], fmaf(k_prev[i], u_prev, s[i]));
+                        rk[e] = fmaf(s[i], kk[i], rk[e]);
+                        rq[e] = fmaf(s[i], qq[i], rq[e]);
+                        kq[e] = fmaf(kk[i], qq[i], kq[e]);
+                    }
+                }
+                float r = (rk[0] + rk[1]) + (rk[2] + rk[3]);
+                float w = (rq[0] + rq[1]) + (rq[2] + rq[3]);
+                float c = (kq[0] + kq[1]) + (kq[2] + kq[3]);
+#pragma unroll
+                for (int x = 1; x < LANES; x <<= 1) {
+                    r += __shfl_xor_sync(0xffffffffu, r, x);
+                    w += __shfl_xor_sync(0xffffffffu, w, x);
+                    c += __shfl_xor_sync(0xffffffffu, c, x);
+                }
+                const float u = beta * (v - r);
+                if (live && part == 0) out[out_at] = fmaf(u, c, w);
+#pragma unroll
+                for (int i = 0; i < P; ++i) k_prev[i] = kk[i];
                 u_prev = u;
             } else if (RULE == RULE_WKV || RULE == RULE_SSD) {
                 // As below: the update needs no sum over a column; a token's sum is reduced and
@@ -439,6 +612,9 @@ __global__ void __launch_bounds__(THREADS) matrix_memory_kernel(
     if (RULE == RULE_DELTA) {
 #pragma unroll
         for (int i = 0; i < P; ++i) s[i] = fmaf(k_prev[i], u_prev, g_prev * s[i]);      // the last token's write
+    } else if (RULE == RULE_CHANNEL) {
+#pragma unroll
+        for (int i = 0; i < P; ++i) s[i] = fmaf(k_prev[i], u_prev, s[i]);
     } else if ((RULE == RULE_WKV || RULE == RULE_SSD) && pending) {
 #pragma unroll
         for (int x = 1; x < LANES; x <<= 1) p_o += __shfl_xor_sync(0xffffffffu, p_o, x);
@@ -582,10 +758,10 @@ __global__ void gate_group_norm_kernel(const float* __restrict__ y, const T* __r
 // ---- per-head RMS norm, gain and output gate ----------------------------------------------
 // o: fp32 [rows][H*E].  gain: [E] shared by the heads (gain_head_stride 0) or [H*E], or null
 // (a norm without a weight).
-// gate: T rows (the joint projection) at a column offset.  out: T rows at a column offset.
-template <typename T, int GATE>
+// gate: rows of TG (columns of the joint projection in T, or fp32).  out: T rows at a column offset.
+template <typename T, typename TG, int GATE>
 __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* __restrict__ gain,
-                                      int gain_head_stride, const T* __restrict__ gate, int gate_stride,
+                                      int gain_head_stride, const TG* __restrict__ gate, int gate_stride,
                                       T* __restrict__ out, int out_stride, int n_rows, int n_heads,
                                       int E, float eps, float out_scale) {
     cb_pdl_trigger();
@@ -598,7 +774,7 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, const float* 
     float ss = 0.f;
     for (int e = lane; e < E; e += 32) ss = fmaf(src[e], src[e], ss);
     const float r = 1.0f / sqrtf(cb_warp_sum(ss) / (float)E + eps);
-    const T* grow = gate + (size_t)t * gate_stride + (size_t)h * E;
+    const TG* grow = gate + (size_t)t * gate_stride + (size_t)h * E;
     T* dst = out + (size_t)t * out_stride + (size_t)h * E;
     const float* gn = gain != nullptr ? gain + (size_t)h * gain_head_stride : nullptr;
     for (int e = lane; e < E; e += 32) {
@@ -615,14 +791,14 @@ int launch_memory_as(const float* qkv, int C, int q_off, int k_off, int v_off, c
                      unsigned char* state, long slot_stride, long s_off, long n_off, long m_off, float* out,
                      int n_requests, int n_heads, int n_qk_heads, int D, int E, int w_off,
                      const float* per_head, cudaStream_t s) {
-    constexpr int COLS = THREADS / LANES, PAD = P == 4 ? 8 : 4, NVEC = RULE == RULE_WKV ? 3 : 2;
+    constexpr int COLS = THREADS / LANES, PAD = P == 4 ? 8 : 4, NVEC = VECTOR_DECAY<RULE> ? 3 : 2;
     const dim3 grid(n_requests, n_heads, (E + COLS - 1) / COLS), block(THREADS);
     const size_t smem = 2 * (size_t)(CHUNK * (NVEC * LANES * (P + PAD) + COLS) + 2 * CHUNK) * sizeof(float);
     if (smem > 48 * 1024) {
         static bool configured = false;
         if (!configured) {
             cudaError_t e = cudaFuncSetAttribute(matrix_memory_kernel<P, LANES, RULE>,
-                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, 100 * 1024);
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
             if (e != cudaSuccess) return (int)e;
             configured = true;
         }
@@ -681,6 +857,37 @@ CB_EXPORT int cb_delta_prepare(const void* proj, int proj_stride, int dtype, con
                   proj_stride, conv_w, taps, gates, gates_stride, a_log, dt_bias, row_request, req_row_start,
                   req_state_slot, (unsigned char*)state, slot_stride, tail_off, qkv, beta, decay,
                   n_heads, n_kv_heads, key_dim, value_dim);
+    return cb_last_error();
+}
+
+// conv_w: fp32 [taps][channels]; max_new: the most tokens that a request brings.
+CB_EXPORT int cb_channel_delta_prepare(const void* proj, int proj_stride, int dtype, const float* conv_w,
+                                       int taps, const float* rate, int rate_stride, const float* beta_logit,
+                                       int beta_stride, const float* a_log, const float* dt_bias,
+                                       const int* req_row_start, const int* req_state_slot, void* state,
+                                       long slot_stride, long tail_off, float* qkv, float* beta,
+                                       int n_requests, int max_new, int H, int G, int D, int E, void* stream) {
+    if (n_requests <= 0 || max_new <= 0) return 0;
+    if (taps < 1 || taps > 64 || H % G != 0 || D > 256 || n_requests > 65535) return CB_ERR_UNSUPPORTED;
+    const int n_units = 2 * G + (H * E + CHANNEL_RUN - 1) / CHANNEL_RUN + (H * D + CHANNEL_RUN - 1) / CHANNEL_RUN + 1;
+    const int tile = taps - 1 > CHANNEL_TILE ? taps - 1 : CHANNEL_TILE;      // a later tile never reads the state
+    const dim3 grid((n_units + 3) / 4, (max_new + tile - 1) / tile, n_requests), block(128);
+    if (grid.y > 65535) return CB_ERR_UNSUPPORTED;
+    cudaStream_t s = (cudaStream_t)stream;
+#define CB_CDP(TT, KK)                                                                                      \
+    cb_launch(channel_delta_prepare_kernel<TT, KK>, grid, block, 0, s, (const TT*)proj, proj_stride, conv_w, \
+              taps, rate, rate_stride, beta_logit, beta_stride, a_log, dt_bias, req_row_start,              \
+              req_state_slot, (unsigned char*)state, slot_stride, tail_off, qkv, beta, H, G, D, E, n_units, tile)
+#define CB_CDP_TAPS(TT)                                                                                     \
+    do {                                                                                                    \
+        if (taps == 2) CB_CDP(TT, 2);                                                                       \
+        else if (taps == 3) CB_CDP(TT, 3);                                                                  \
+        else if (taps == 4) CB_CDP(TT, 4);                                                                  \
+        else CB_CDP(TT, 0);                                                                                 \
+    } while (0)
+    if (dtype == CB_F32) CB_CDP_TAPS(float); else CB_CDP_TAPS(__nv_bfloat16);
+#undef CB_CDP_TAPS
+#undef CB_CDP
     return cb_last_error();
 }
 
@@ -743,7 +950,8 @@ CB_EXPORT int cb_retention_prepare(const void* proj, int proj_stride, int dtype,
 
 // rule 0: the delta rule (sc0 decay, sc1 beta); rule 1: mLSTM (sc0 log keep, sc1 log in);
 // rule 2: wkv (decay vectors at w_off in the rows, per_head the bonus [H][D]);
-// rule 3: state space (sc0 decay, sc1 step size, per_head the skip [H]).
+// rule 3: state space (sc0 decay, sc1 step size, per_head the skip [H]);
+// rule 4: channel delta (decay vectors at w_off, one of D per head; sc1 beta).
 CB_EXPORT int cb_matrix_memory(int rule, const float* qkv, int C, int q_off, int k_off, int v_off,
                                const float* sc0, const float* sc1, const int* req_row_start,
                                const int* req_state_slot, void* state, long slot_stride, long s_off,
@@ -764,28 +972,34 @@ CB_EXPORT int cb_matrix_memory(int rule, const float* qkv, int C, int q_off, int
     CB_RULE(RULE_MLSTM);
     CB_RULE(RULE_WKV);
     CB_RULE(RULE_SSD);
+    CB_RULE(RULE_CHANNEL);
 #undef CB_RULE
     return CB_ERR_UNSUPPORTED;
 }
 
 // gate_kind 0: SiLU, 1: sigmoid.
 CB_EXPORT int cb_head_norm_gate(const float* o, const float* gain, int gain_head_stride,
-                                const void* gate, int gate_stride, void* out, int out_stride, int dtype,
-                                int gate_kind, int n_rows, int n_heads, int value_dim, float eps,
+                                const void* gate, int gate_stride, int gate_dtype, void* out, int out_stride,
+                                int dtype, int gate_kind, int n_rows, int n_heads, int value_dim, float eps,
                                 float out_scale, void* stream) {
     if (n_rows <= 0) return 0;
     const int warps = 4;
     const long units = (long)n_rows * n_heads;
     const dim3 grid((unsigned)((units + warps - 1) / warps)), block(warps * 32);
     cudaStream_t s = (cudaStream_t)stream;
-#define CB_HNG(TT, GG)                                                                             \
-    cb_launch(head_norm_gate_kernel<TT, GG>, grid, block, 0, s, o, gain, gain_head_stride,         \
-              (const TT*)gate, gate_stride, (TT*)out, out_stride, n_rows, n_heads, value_dim, eps, \
+#define CB_HNG(TT, TGG, GG)                                                                        \
+    cb_launch(head_norm_gate_kernel<TT, TGG, GG>, grid, block, 0, s, o, gain, gain_head_stride,    \
+              (const TGG*)gate, gate_stride, (TT*)out, out_stride, n_rows, n_heads, value_dim, eps, \
               out_scale)
     if (dtype == CB_F32) {
-        if (gate_kind == GATE_SILU) CB_HNG(float, GATE_SILU); else CB_HNG(float, GATE_SIGMOID);
+        if (gate_dtype != CB_F32) return CB_ERR_UNSUPPORTED;
+        if (gate_kind == GATE_SILU) CB_HNG(float, float, GATE_SILU); else CB_HNG(float, float, GATE_SIGMOID);
+    } else if (gate_dtype == CB_F32) {
+        if (gate_kind == GATE_SILU) CB_HNG(__nv_bfloat16, float, GATE_SILU);
+        else CB_HNG(__nv_bfloat16, float, GATE_SIGMOID);
     } else {
-        if (gate_kind == GATE_SILU) CB_HNG(__nv_bfloat16, GATE_SILU); else CB_HNG(__nv_bfloat16, GATE_SIGMOID);
+        if (gate_kind == GATE_SILU) CB_HNG(__nv_bfloat16, __nv_bfloat16, GATE_SILU);
+        else CB_HNG(__nv_bfloat16, __nv_bfloat16, GATE_SIGMOID);
     }
 #undef CB_HNG
     return cb_last_error();

@@ -16,7 +16,8 @@
 //     position with a running maximum, fp32 throughout.  A row at position p sees
 //     j <= p with p - j < window or j < keep_first, i.e. the ranges
 //     [0, min(keep_first, lo)) and [lo, p], lo = max(0, p - window + 1); window 0
-//     means every earlier key.  After the keys the sink joins the denominator:
+//     means every earlier key; `chunked`: the window is the size of chunks counted from
+//     position 0 and lo is the first position of the row's chunk.  After the keys the sink joins the denominator:
 //     l += exp(sink[h] - m), with no value.  With a gate, the head's result is
 //     multiplied by sigmoid(gate) and by out_scale before it is stored.
 // A row's result depends on its own query and keys only.
@@ -209,7 +210,7 @@ __global__ void sink_attention_kernel(
     const float* __restrict__ sinks, const int* __restrict__ positions,
     const int* __restrict__ row_request, const int* __restrict__ block_table, int table_stride,
     int n_rows, int n_heads, int n_kv_heads, int key_dim, int value_dim, int page_tokens,
-    float scale, int window, int keep_first, float out_scale, int gate_per_head) {
+    float scale, int window, int chunked, int keep_first, float out_scale, int gate_per_head) {
     cb_pdl_trigger();
     cb_pdl_wait();
     const int warps_per_block = blockDim.x >> 5;
@@ -220,7 +221,7 @@ __global__ void sink_attention_kernel(
     const int kvh = h / (n_heads / n_kv_heads);
     const int pos = positions[t];
     const int* table = block_table + (size_t)row_request[t] * table_stride;
-    const int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
+    const int lo = window <= 0 ? 0 : chunked ? pos - pos % window : max(0, pos - window + 1);
     const int kept = keep_first < lo ? keep_first : lo;      // keys [0, kept) and [lo, pos]
 
     float qv[MAX_PER_LANE], acc[MAX_PER_LANE];
@@ -343,7 +344,7 @@ CB_EXPORT int cb_sink_attention(const void* q, int q_stride, const void* gate, i
                                 int dtype, const float* sinks, const int* positions,
                                 const int* row_request, const int* block_table, int table_stride,
                                 int n_rows, int n_heads, int n_kv_heads, int key_dim, int value_dim,
-                                int page_tokens, float scale, int window, int keep_first,
+                                int page_tokens, float scale, int window, int chunked, int keep_first,
                                 float out_scale, int gate_per_head, void* stream) {
     if (n_rows <= 0) return 0;
     if (key_dim > 1024 || value_dim > 1024 || n_heads % n_kv_heads != 0) return CB_ERR_UNSUPPORTED;
@@ -356,7 +357,7 @@ CB_EXPORT int cb_sink_attention(const void* q, int q_stride, const void* gate, i
     cb_launch(sink_attention_kernel<TT, PL>, dim3(blocks), dim3(warps * 32), 0, s, (const TT*)q, q_stride, \
               (const TT*)gate, gate_stride, (TT*)out, out_stride, (const TT*)k_cache, (const TT*)v_cache, \
               sinks, positions, row_request, block_table, table_stride, n_rows, n_heads, n_kv_heads,    \
-              key_dim, value_dim, page_tokens, scale, window, keep_first, out_scale, gate_per_head)
+              key_dim, value_dim, page_tokens, scale, window, chunked, keep_first, out_scale, gate_per_head)
     if (dtype == CB_F32) {
         if (wide) CB_SINK_LAUNCH(float, 32);
         else CB_SINK_LAUNCH(float, 8);

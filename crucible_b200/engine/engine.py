@@ -152,7 +152,7 @@ class Engine:
         # refused before anything is written (`engine/src/gpu_model.rs:2809-2934` refuses
         # such a batch).
         self.cache = CacheManager(
-            [GroupPolicy(o.page_tokens, g.need.window, g.need.keep_first) for g in groups],
+            [GroupPolicy(o.page_tokens, g.need.window, g.need.keep_first, g.need.chunked) for g in groups],
             [n_pages] * len(groups), o.max_requests, table_strides=self.table_strides,
             null_pages=[self.null_page] * len(groups))
         self._has_device_token = set()      # state slots whose latest token is on the device

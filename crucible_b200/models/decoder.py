@@ -112,10 +112,12 @@ class DecoderModel:
         for i, entry in enumerate(self.config.run_order):
             layer = self.layers[entry.layer]
             nbytes = int(layer.mixer.state_bytes())
+            own = int(getattr(layer, "own_state_bytes", lambda: 0)())
             me = (entry.layer, entry.copy)
-            if nbytes and me not in state_offsets:
+            if (nbytes or own) and me not in state_offsets:
+                # the mixer's bytes, then the arrangement's own
                 state_offsets[me] = total_state
-                total_state += (nbytes + 15) // 16 * 16
+                total_state += (nbytes + 15) // 16 * 16 + (own + 15) // 16 * 16
             group = slot = None
             write = True
             if entry.cache_of is not None:
@@ -138,13 +140,16 @@ class DecoderModel:
                                       f"time and would write its cache twice; name "
                                       f"cache_of to read it instead, or another copy")
                 written.add(me)
-            elif nbytes and me in ran:
+            if (nbytes or own) and me in ran:
                 raise ConfigError(f"run_order[{i}] runs layer {entry.layer} a second time on "
                                   f"the same state; name another copy")
             ran.add(me)
             bindings.append(LayerBinding(group=group, slot=slot or 0, write=write,
                                          state_offset=state_offsets.get(me, 0),
-                                         state_bytes=nbytes))
+                                         state_bytes=nbytes,
+                                         own=LayerBinding(
+                                             state_offset=state_offsets[me] + (nbytes + 15) // 16 * 16,
+                                             state_bytes=own) if own else None))
         specs = [CacheGroupSpec(need, tuple(members)) for need, members in groups]
         return specs, bindings, total_state
 
@@ -190,6 +195,11 @@ class DecoderModel:
             part.bind(mine, dtype, device)
         if self.config.tie_word_embeddings:
             self.head.tie(self.embedding.table)
+        # a head that scales its logits does so by the gain of the norm its rows come from (a
+        # float32 number on the rows before they are rounded)
+        scale = float(getattr(self.head, "scale", 1.0))
+        if scale != 1.0:
+            self.final_norm.scale_gain(scale)
 
     @property
     def graph_safe(self) -> bool:
@@ -219,15 +229,22 @@ class DecoderModel:
         """Runs the step's tokens; returns fp32 logits [wanted rows, vocab]."""
         x = self.embedding.forward(ctx, ctx.token_ids)
         order = self.config.run_order
+        embedded = None
+        if any(entry.add_embedding for entry in order):
+            embedded = ctx.scratch("embedding.output", x.shape, torch.float32)
+            embedded.copy_(x)
         for i, (entry, binding) in enumerate(zip(order, self.bindings)):
             # the norm that reads the rows after this layer, for the layer's last product
             nxt = self.layers[order[i + 1].layer] if i + 1 < len(order) else None
             entry_norm = getattr(nxt, "entry_norm", None)
             # (rows that get a vector added before the next layer are not final when this one ends)
-            ctx.norm_after_layer = (entry_norm() if entry_norm is not None and order[i + 1].add is None
-                                    else None)
-            if entry.add is not None:
-                ops.add_vector(x, self.vectors.row(*entry.add))
+            changed = i + 1 < len(order) and (order[i + 1].add is not None or order[i + 1].add_embedding)
+            ctx.norm_after_layer = entry_norm() if entry_norm is not None and not changed else None
+            vector = self.vectors.row(*entry.add) if entry.add is not None else None
+            if entry.add_embedding:
+                ops.add_rows(x, embedded, vector)
+            elif vector is not None:
+                ops.add_vector(x, vector)
             self.layers[entry.layer].forward(ctx, x, binding)
         ctx.norm_after_layer = None
         if ctx.n_logit_rows == 0:

@@ -30,10 +30,9 @@ from collections.abc import Mapping as _Mapping
 from typing import Any, Mapping
 
 from ..config.model_config import (UNBOUNDED_CONTEXT, ConfigError, EndSpec, FeedForwardSpec, KeyReader,
-                                   LayerSpec, MixerSpec, ModelConfig, NormSpec, PositionSpec, RunEntry)
+                                   LayerSpec, MixerSpec, ModelConfig, NormSpec, PositionSpec)
 from ..config.registry import Architecture, register_architecture
-
-LOOP_VECTORS = "loop_step"      # the model's table of the vectors added before each pass
+from .loops import LOOP_VECTORS, looped_run_order
 
 
 class _Names(_Mapping):
@@ -138,30 +137,6 @@ def _feed_forward(mlp, width: int, where: str) -> FeedForwardSpec:
                            extra=(("activation", "relu2"),))
 
 
-def _run_order(raw, n_layers: int):
-    """(run order, rows of the passes' vectors): the looped layers once per pass, each pass a
-    copy with keys and state of its own; the pass's vector is added before its first layer."""
-    loop = raw.get("loop")
-    if loop is None:
-        return tuple(RunEntry(layer=i) for i in range(n_layers)), 0
-    where = "config.json loop"
-    if not isinstance(loop, dict):
-        raise ConfigError(f"{where}: must be an object")
-    start, stop = _count(loop, "start", where), _count(loop, "stop", where)
-    times = KeyReader(loop, where).integer("times")
-    if not start <= stop <= n_layers:
-        raise ConfigError(f"{where}: 'start' <= 'stop' <= the number of layers, got {start} and {stop}")
-    if start == stop:
-        # an empty run: nothing repeats and no vector is ever added (the table is still the model's)
-        return tuple(RunEntry(layer=i) for i in range(n_layers)), times
-    order = [RunEntry(layer=i) for i in range(start)]
-    for t in range(times):
-        order += [RunEntry(layer=i, copy=t, add=(LOOP_VECTORS, t) if i == start else None)
-                  for i in range(start, stop)]
-    order += [RunEntry(layer=i) for i in range(stop, n_layers)]
-    return tuple(order), times
-
-
 def _parse(raw: Mapping[str, Any]) -> ModelConfig:
     r = KeyReader(raw)
     width, vocab = r.integer("width"), r.integer("vocab")
@@ -186,7 +161,7 @@ def _parse(raw: Mapping[str, Any]) -> ModelConfig:
         layers.append(LayerSpec(arrangement="parallel", mixer=mixer,
                                 feed_forward=_feed_forward(entry.get("mlp"), width, where + ".mlp"),
                                 norms=(("norm", norm),)))
-    order, times = _run_order(raw, len(layers))
+    order, times = looped_run_order(raw, len(layers))
     return ModelConfig(
         architecture="Sebalorn", vocab_size=vocab, hidden_size=width, max_context=UNBOUNDED_CONTEXT,
         tie_word_embeddings=False, layers=tuple(layers), run_order=order, final_norm=norm,

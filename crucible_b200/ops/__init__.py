@@ -239,6 +239,20 @@ def add_vector(x: torch.Tensor, v: torch.Tensor) -> None:
            "add_vector")
 
 
+def add_rows(x: torch.Tensor, rows: torch.Tensor, v: Optional[torch.Tensor] = None) -> None:
+    """x[t, :] += rows[t, :], then += v if given, for every row of the float32 residual."""
+    _need_cuda(x, rows, v)
+    if (x.dtype != torch.float32 or rows.dtype != torch.float32 or x.dim() != 2 or rows.shape != x.shape
+            or (v is not None and (v.dtype != torch.float32 or v.dim() != 1 or v.shape[0] != x.shape[1]))):
+        raise KernelError("add_rows takes float32 rows [T, W] twice and a float32 vector [W]")
+    _contig(x, "add_rows rows"); _contig(rows, "add_rows added rows")
+    if v is not None:
+        _contig(v, "add_rows vector")
+    lib = build.load("elementwise")
+    _check(lib.cb_add_rows(_ptr(x), _ptr(rows), _ptr(v), _c_int(x.shape[0]), _c_int(x.shape[1]), _stream()),
+           "add_rows")
+
+
 def softcap(z: torch.Tensor, cap: float) -> None:
     """z <- cap * tanh(z / cap) in place, float32 rows."""
     _need_cuda(z)

@@ -50,6 +50,8 @@ MODULES: Dict[str, List[str]] = {
     "activations": ["common.cuh"],
     "latent_attention": ["common.cuh"],
     "moe": ["common.cuh"],
+    "input_conv": ["common.cuh"],
+    "differential": ["common.cuh"],
 }
 
 _loaded: Dict[str, ctypes.CDLL] = {}

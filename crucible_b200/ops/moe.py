@@ -33,24 +33,35 @@ def _pair(pair):
 
 
 def route(logits, top: int, idx, weight, place, count, plan, tiles: int, sorted_pair, bias=None,
-          rows: int = 0) -> None:
+          rows: int = 0, n_experts: int = 0, groups=None, n_shared: int = 0, gate_col: int = -1,
+          scale: float = 1.0, gate_out=None) -> None:
     """Per token the `top` largest logits (plus `bias`, float32 [experts], if given; the lower
     index on ties) and their softmax; then
     the sorted order of the (token, choice) pairs by expert and the tiles (of `rows` rows; 0: this
     file's own) over it.  `count`
-    (int32 [experts]) is zero between calls: the kernels leave it so."""
-    _need_cuda(logits, idx, weight, place, count, plan, sorted_pair, bias)
+    (int32 [experts]) is zero between calls: the kernels leave it so.
+    `n_experts`: the logits' first columns that are the experts' (0: all).  `groups` = (count, keep):
+    the experts form that many equal groups of neighbours, of which those with the `keep` largest best
+    logits take part.  `n_shared` slices of a shared expert ride along as further experts (after the
+    routed ones) that every token chooses, weighted by the sigmoid of logit `gate_col`; `gate_out`
+    (float32 [tokens] or None) receives that weight.  `scale`: on every weight.  `count` and the plan
+    cover the slices too, and a token has top + n_shared pairs."""
+    _need_cuda(logits, idx, weight, place, count, plan, sorted_pair, bias, gate_out)
     if logits.dtype != torch.float32 or not logits.is_contiguous():
         raise KernelError("moe route takes contiguous float32 logits [tokens, experts]")
-    t, e = logits.shape
+    t, e = logits.shape[0], n_experts or logits.shape[1]
+    pairs, total = t * (top + n_shared), e + n_shared
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != e or not bias.is_contiguous()):
         raise KernelError("moe route: the bias is float32 [experts]")
-    if idx.numel() < t * top or plan.numel() < plan_ints(e, tiles) or sorted_pair.numel() < t * top:
+    if (idx.numel() < pairs or plan.numel() < plan_ints(total, tiles) or sorted_pair.numel() < pairs
+            or count.numel() < total):
         raise KernelError("moe route: a buffer is too small")
     lib = build.load("moe")
-    _check(lib.cb_moe_route(_ptr(logits), _ptr(bias), _c_int(t), _c_int(e), _c_int(top), _ptr(idx), _ptr(weight),
-                            _ptr(place), _ptr(count), _ptr(plan), _c_int(tiles), _ptr(sorted_pair),
-                            _c_int(rows), _stream()), "moe route")
+    count_g, keep_g = groups if groups is not None else (1, 1)
+    _check(lib.cb_moe_route(_ptr(logits), _c_int(logits.shape[1]), _ptr(bias), _c_int(t), _c_int(e), _c_int(top),
+                            _ptr(idx), _ptr(weight), _ptr(place), _ptr(count), _ptr(plan), _c_int(tiles),
+                            _ptr(sorted_pair), _c_int(rows), _c_int(count_g), _c_int(keep_g), _c_int(n_shared),
+                            _c_int(gate_col), ctypes.c_float(scale), _ptr(gate_out), _stream()), "moe route")
 
 
 def expert_tiles(gated: bool, a, w, n_out: int, plan, n_experts: int, tiles: int, sorted_pair, top: int,
@@ -91,14 +102,21 @@ def expert_rows_small(gated: bool, a, w, n_out: int, plan, n_experts: int, tiles
     return True
 
 
-def combine(pair_out, top: int, residual) -> None:
-    """residual[t] += sum over the token's choices, in their order."""
-    _need_cuda(pair_out, residual)
-    if pair_out.dtype != torch.float32 or residual.dtype != torch.float32 or not residual.is_contiguous():
+def combine(rows, top: int, residual, by_plan=None, shared=None, gate=None) -> None:
+    """residual[t] += sum over the token's choices, in their order.  `rows` lie pair by pair and
+    weighted, or, with `by_plan` = (plan, idx, place, weight) of `route`, in the sorted order and are
+    weighted here.  `shared` (float32 rows by token) joins with `gate` (float32 [tokens])."""
+    plan, idx, place, weight = by_plan if by_plan is not None else (None,) * 4
+    _need_cuda(rows, residual, plan, idx, place, weight, shared, gate)
+    if (rows.dtype != torch.float32 or residual.dtype != torch.float32 or not residual.is_contiguous()
+            or not rows.is_contiguous() or (shared is None) != (gate is None)
+            or (shared is not None and (shared.dtype != torch.float32 or shared.shape != residual.shape
+                                        or not shared.is_contiguous() or gate.dtype != torch.float32))):
         raise KernelError("moe combine adds float32 rows into the float32 residual")
     lib = build.load("moe")
-    _check(lib.cb_moe_combine(_ptr(pair_out), _c_int(top), _ptr(residual), _c_int(residual.shape[0]),
-                              _c_int(residual.shape[1]), _stream()), "moe combine")
+    _check(lib.cb_moe_combine(_ptr(rows), _c_int(top), _ptr(residual), _c_int(residual.shape[0]),
+                              _c_int(residual.shape[1]), _ptr(plan), _ptr(idx), _ptr(place), _ptr(weight),
+                              _ptr(shared), _ptr(gate), _stream()), "moe combine")
 
 
 def gather(h, sorted_pair, top: int, out) -> None:
@@ -108,14 +126,6 @@ def gather(h, sorted_pair, top: int, out) -> None:
     _check(lib.cb_moe_gather(_ptr(h), _c_int(h.stride(0)), _c_int(_code(h.dtype)), _ptr(sorted_pair),
                              _c_int(top), _ptr(out), _c_int(out.shape[0]), _c_int(h.shape[1]), _stream()),
            "moe gather")
-
-
-def scatter(rows, sorted_pair, weight, pair_out) -> None:
-    """pair_out[pair] = weight[pair] * rows[the pair's sorted place]."""
-    _need_cuda(rows, sorted_pair, weight, pair_out)
-    lib = build.load("moe")
-    _check(lib.cb_moe_scatter(_ptr(rows), _ptr(sorted_pair), _ptr(weight), _ptr(pair_out),
-                              _c_int(rows.shape[0]), _c_int(rows.shape[1]), _stream()), "moe scatter")
 
 
 def grouped_linear(rows_sorted, w, out, plan, n_experts: int, tiles: int, gated: bool, pair=None) -> bool:

@@ -1,6 +1,6 @@
 """Wrappers of `csrc/recurrent.cu`: mixers that carry a matrix per head from token to
 token in the request's state slot (the gated delta rule, the mLSTM, the wkv rule, the
-state-space rule)."""
+state-space rule, the delta rule with a decay per key channel)."""
 from __future__ import annotations
 
 import ctypes
@@ -10,7 +10,7 @@ import torch
 from . import KernelError, _c_float, _c_int, _check, _code, _need_cuda, _ptr, _stream, build
 
 _c_long = ctypes.c_long
-DELTA, MLSTM, WKV, SSD = 0, 1, 2, 3
+DELTA, MLSTM, WKV, SSD, CHANNEL = 0, 1, 2, 3, 4
 GATE_SILU, GATE_SIGMOID = 0, 1
 
 
@@ -33,6 +33,32 @@ def delta_prepare(proj, conv_w, taps, gates, a_log, dt_bias, ctx, state, tail_of
         _ptr(ctx.req_state_slot), sp, stride, _c_long(tail_off), _ptr(qkv), _ptr(beta), _ptr(decay),
         _c_int(proj.shape[0]), _c_int(n_heads), _c_int(n_kv_heads), _c_int(key_dim),
         _c_int(value_dim), _stream()), "delta_prepare")
+
+
+def channel_delta_prepare(proj, conv_w, rate, beta_logit, a_log, dt_bias, ctx, state, tail_off, qkv, beta,
+                          n_heads, n_qk_heads, key_dim, value_dim) -> None:
+    """`proj` rows [q: G*D | k: G*D | v: H*E | ...], `conv_w` float32 [taps, channels], `rate`
+    float32 rows of H*D decay logits, `beta_logit` float32 rows of H.  qkv = float32
+    [unit q * D^-1/2 | unit k | v | exp(-exp(a_log) softplus(rate + dt_bias))], beta = sigmoid; the
+    convolution's inputs in the state (float32 [taps - 1, channels] at `tail_off`) are read and
+    rewritten."""
+    _need_cuda(proj, conv_w, rate, beta_logit, a_log, dt_bias, state, qkv, beta)
+    C = 2 * n_qk_heads * key_dim + n_heads * value_dim
+    f32 = torch.float32
+    if (proj.stride(1) != 1 or proj.shape[1] < C or conv_w.dtype != f32 or not conv_w.is_contiguous()
+            or conv_w.shape[1] != C or rate.dtype != f32 or rate.stride(1) != 1 or rate.shape[1] < n_heads * key_dim
+            or beta_logit.dtype != f32 or beta_logit.stride(1) != 1 or qkv.dtype != f32 or not qkv.is_contiguous()
+            or qkv.shape[1] != C + n_heads * key_dim or beta.dtype != f32 or not beta.is_contiguous()
+            or a_log.numel() != n_heads or dt_bias.numel() != n_heads * key_dim):
+        raise KernelError("channel_delta_prepare: rows [q | k | v], float32 taps [taps, channels], logits and outputs")
+    sp, stride = _state_args(state)
+    lib = build.load("recurrent")
+    _check(lib.cb_channel_delta_prepare(
+        _ptr(proj), _c_int(proj.stride(0)), _c_int(_code(proj.dtype)), _ptr(conv_w), _c_int(conv_w.shape[0]),
+        _ptr(rate), _c_int(rate.stride(0)), _ptr(beta_logit), _c_int(beta_logit.stride(0)), _ptr(a_log),
+        _ptr(dt_bias), _ptr(ctx.req_row_start), _ptr(ctx.req_state_slot), sp, stride, _c_long(tail_off), _ptr(qkv),
+        _ptr(beta), _c_int(ctx.n_requests), _c_int(ctx.host.max_new_tokens), _c_int(n_heads), _c_int(n_qk_heads),
+        _c_int(key_dim), _c_int(value_dim), _stream()), "channel_delta_prepare")
 
 
 def conv_tail_update(proj, taps, channels, ctx, state, tail_off) -> None:
@@ -82,7 +108,7 @@ def retention_prepare(proj, freq, rotary_dim: int, split_halves: bool, ctx, head
 def matrix_memory(rule, qkv, q_off, k_off, v_off, sc0, sc1, ctx, state, s_off, n_off, m_off, out,
                   n_heads, n_qk_heads, key_dim, value_dim, w_off=0, per_head=None) -> None:
     """Walks every request's tokens in order through its heads' matrices (see the kernel).
-    `w_off`: where the wkv rule's decay vectors lie in the rows of `qkv`; `per_head`: float32
+    `w_off`: where the wkv and channel rules' decay vectors (one a head) lie in the rows of `qkv`; `per_head`: float32
     constants, the wkv rule's bonus [heads, key_dim] or the state-space rule's skip [heads]."""
     _need_cuda(qkv, sc0, sc1, state, out, per_head)
     if per_head is not None and (per_head.dtype != torch.float32 or not per_head.is_contiguous()):
@@ -101,16 +127,17 @@ def matrix_memory(rule, qkv, q_off, k_off, v_off, sc0, sc1, ctx, state, s_off, n
 
 def head_norm_gate(o, gain, gain_per_head, gate, out, gate_kind, n_heads, value_dim, eps,
                    out_scale) -> None:
-    """out = o / rms(o over a head) * gain * act(gate) * out_scale; `gate` and `out` are
-    views of rows in the engine dtype.  `gain` None: a norm without a weight."""
+    """out = o / rms(o over a head) * gain * act(gate) * out_scale; `out` is a view of rows in
+    the engine dtype, `gate` one in the engine dtype or in float32.  `gain` None: a norm without a weight."""
     _need_cuda(o, gain, gate, out)
-    if o.dtype != torch.float32 or gate.dtype != out.dtype or gate.stride(1) != 1 or out.stride(1) != 1:
-        raise KernelError("head_norm_gate: float32 input, gate and output rows of one dtype")
+    if (o.dtype != torch.float32 or gate.dtype not in (out.dtype, torch.float32) or gate.stride(1) != 1
+            or out.stride(1) != 1):
+        raise KernelError("head_norm_gate: float32 input, gate rows of the output's dtype or float32")
     lib = build.load("recurrent")
     _check(lib.cb_head_norm_gate(
         _ptr(o), _ptr(gain), _c_int(value_dim if gain_per_head else 0), _ptr(gate),
-        _c_int(gate.stride(0)), _ptr(out), _c_int(out.stride(0)), _c_int(_code(out.dtype)),
-        _c_int(gate_kind), _c_int(o.shape[0]), _c_int(n_heads), _c_int(value_dim), _c_float(eps),
+        _c_int(gate.stride(0)), _c_int(_code(gate.dtype)), _ptr(out), _c_int(out.stride(0)),
+        _c_int(_code(out.dtype)), _c_int(gate_kind), _c_int(o.shape[0]), _c_int(n_heads), _c_int(value_dim), _c_float(eps),
         _c_float(out_scale), _stream()), "head_norm_gate")
 
 

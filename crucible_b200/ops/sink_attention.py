@@ -77,9 +77,11 @@ def norm_rotate_append(proj: torch.Tensor, q_gain: Optional[torch.Tensor], k_gai
 def attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
               sinks: Optional[torch.Tensor], n_heads: int, n_kv_heads: int, key_dim: int,
               value_dim: int, scale: float, window: Optional[int], keep_first: int,
-              out_scale: float, ctx, cache, binding, gate_per_head: bool = False) -> None:
+              out_scale: float, ctx, cache, binding, gate_per_head: bool = False,
+              chunked: bool = False) -> None:
     """`q`, `gate`, `out`: views of rows (unit stride along features).  Position p sees
-    j <= p with p - j < window or j < keep_first.  out = softmax-with-sink(q k) v, times
+    j <= p with p - j < window or j < keep_first; with `chunked` the window is the size of chunks
+    counted from position 0 and p sees j <= p of its own chunk.  out = softmax-with-sink(q k) v, times
     sigmoid(gate) if given, times out_scale.  `gate`: rows laid out like `out` (a logit for
     every feature), or [rows, n_heads] with `gate_per_head` (one logit a head)."""
     _need_cuda(q, gate, out, sinks)
@@ -93,7 +95,7 @@ def attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
     if gate is not None and gate.dtype != q.dtype:
         raise KernelError("sink attention: the gate's logits are rows of the queries' dtype")
     if _tensor_cores(q, gate, out, sinks, n_heads, n_kv_heads, key_dim, value_dim, scale, window,
-                     keep_first, out_scale, ctx, cache, k_cache, v_cache, table, gate_per_head):
+                     keep_first, out_scale, ctx, cache, k_cache, v_cache, table, gate_per_head, chunked):
         return
     lib = build.load("sink_attention")
     _check(lib.cb_sink_attention(
@@ -101,32 +103,34 @@ def attention(q: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
         _ptr(out), _c_int(out.stride(0)), _ptr(k_cache), _ptr(v_cache), _c_int(_code(q.dtype)),
         _ptr(sinks), _ptr(ctx.positions), _ptr(ctx.row_request), _ptr(table), _c_int(table.shape[1]),
         _c_int(q.shape[0]), _c_int(n_heads), _c_int(n_kv_heads), _c_int(key_dim), _c_int(value_dim),
-        _c_int(cache.page_tokens), _c_float(scale), _c_int(window or 0), _c_int(keep_first),
-        _c_float(out_scale), _c_int(1 if gate_per_head else 0), _stream()), "sink attention")
+        _c_int(cache.page_tokens), _c_float(scale), _c_int(window or 0), _c_int(1 if chunked else 0),
+        _c_int(keep_first), _c_float(out_scale), _c_int(1 if gate_per_head else 0), _stream()), "sink attention")
 
 
 TENSOR_CORES = True      # tests switch it off to reach the plain kernel with the same inputs
 
 
 def _tensor_cores(q, gate, out, sinks, n_heads, n_kv_heads, key_dim, value_dim, scale, window,
-                  keep_first, out_scale, ctx, cache, k_cache, v_cache, table, gate_per_head=False) -> bool:
-    """For bfloat16 rows whose keys and values have one size: steps of prompts' portions alone
-    with plain softmax and heads of 64 or 128 take the tcgen05 attention (`csrc/attention_tcgen05.cu`);
-    everything else of a size that is a multiple of 16 up to 256 the mma.sync kernel of 64-row
+                  keep_first, out_scale, ctx, cache, k_cache, v_cache, table, gate_per_head=False,
+                  chunked=False) -> bool:
+    """For bfloat16 rows: steps of prompts' portions alone whose keys and values have one size, 64
+    or 128, without a gate per feature take the tcgen05 attention (`csrc/attention_tcgen05.cu`);
+    everything else of key and value sizes that are multiples of 16 up to 256 the mma.sync kernel of 64-row
     tiles (`csrc/attention_mma.cu`, its extended form): prompts' portions and decoded tokens in
     one launch, the rows of a request's query heads that share a key/value head packed into
     tiles.  Refuses anything else."""
     host = getattr(ctx, "host", None)
-    if (not TENSOR_CORES or q.dtype != torch.bfloat16 or key_dim != value_dim or key_dim % 16
-            or key_dim > 256 or host is None or q.stride(0) % 8 or out.stride(0) % 2
+    if (not TENSOR_CORES or q.dtype != torch.bfloat16 or key_dim % 16 or value_dim % 16
+            or key_dim > 256 or value_dim > 256 or host is None or q.stride(0) % 8 or out.stride(0) % 2
             or (gate is not None and not gate_per_head and gate.stride(0) % 2)):
         return False
     from . import tensor_core
-    # a plain softmax over keys and values of 64 or 128 features, portions of prompts only: the
-    # tcgen05 attention, whose tiles take the kept first tokens ahead of the window's
-    if (sinks is None and (gate is None or gate_per_head) and out_scale == 1.0
+    # keys and values of 64 or 128 features, portions of prompts only: the tcgen05 attention, whose
+    # tiles take the kept first tokens ahead of the window's
+    if (key_dim == value_dim and (gate is None or gate_per_head)
             and tensor_core.prompt_attention(q, out, k_cache, v_cache, n_heads, n_kv_heads, key_dim, scale,
-                                             window, keep_first, ctx, cache, table)):
+                                             window, keep_first, ctx, cache, table, chunked=chunked, sinks=sinks,
+                                             out_scale=out_scale)):
         if gate is not None:
             # one logit a head: a pass over the heads' results behind the attention
             from . import latent
@@ -144,15 +148,15 @@ def _tensor_cores(q, gate, out, sinks, n_heads, n_kv_heads, key_dim, value_dim, 
         n_chunks = max(1, min(tiles // 2, 296 // max(1, n_kv_heads * ctx.n_requests), 32))
         if n_chunks > 1:
             partial = ctx.scratch("sink_attention.partial",
-                                  (ctx.n_requests * n_kv_heads * n_chunks * max_rows * (key_dim + 2),),
+                                  (ctx.n_requests * n_kv_heads * n_chunks * max_rows * (value_dim + 2),),
                                   torch.float32)
     code = lib.cb_attention_mma_sink(
         _ptr(q), _c_int(q.stride(0)), _ptr(out), _c_int(out.stride(0)), _ptr(gate),
         _c_int(gate.stride(0) if gate is not None else 0), _ptr(k_cache), _ptr(v_cache), _ptr(sinks),
         _ptr(ctx.req_row_start), _ptr(ctx.req_first_pos), _ptr(table), _c_int(table.shape[1]),
         _c_int(ctx.n_requests), _c_int(host.max_new_tokens), _c_int(n_heads), _c_int(n_kv_heads),
-        _c_int(key_dim), _c_int(cache.page_tokens), _c_float(scale), _c_int(window or 0),
-        _c_int(keep_first), _c_float(out_scale), _ptr(partial), _c_int(n_chunks),
+        _c_int(key_dim), _c_int(value_dim), _c_int(cache.page_tokens), _c_float(scale), _c_int(window or 0),
+        _c_int(1 if chunked else 0), _c_int(keep_first), _c_float(out_scale), _ptr(partial), _c_int(n_chunks),
         _c_int(1 if gate_per_head else 0), _stream())
     if code == 100001:
         return False

@@ -494,10 +494,11 @@ class _Requests:
 
 
 def _attention_tcgen05(qkv, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, head_dim, scale,
-                       window, cache, keep_first: int = 0) -> bool:
+                       window, cache, keep_first: int = 0, chunked: bool = False, sinks=None, out_scale: float = 1.0) -> bool:
     """tcgen05 attention for portions of prompts: head size 64 or 128, page size a
     power of two from 8 to 128.  `keep_first` (with a window): keys before that position stay
-    visible.  Returns False for anything else."""
+    visible.  `chunked`: the window is a chunk's size.  `sinks`: float32 per query head or None.
+    Returns False for anything else."""
     pt = cache.page_tokens
     if pt < 8 or pt > 128 or pt & (pt - 1):
         return False
@@ -509,8 +510,8 @@ def _attention_tcgen05(qkv, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, he
         _c_void_p(reqs.first_pos.data_ptr()), _c_void_p(reqs.table.data_ptr()),
         _c_int(reqs.table_stride), _c_int(reqs.count), _c_int(reqs.max_new),
         _c_int(n_heads), _c_int(n_kv_heads), _c_int(head_dim), _c_int(pt),
-        ctypes.c_float(scale), _c_int(window or 0), _c_int(keep_first if window else 0), _c_int(ATTENTION_LEAN),
-        _c_void_p(status_word(qkv.device).data_ptr()), _stream())
+        ctypes.c_float(scale), _c_int(window or 0), _c_int(1 if chunked else 0), _c_int(keep_first if window else 0),
+        ctypes.c_float(out_scale), _c_void_p(sinks.data_ptr() if sinks is not None else 0), _c_int(ATTENTION_LEAN), _c_void_p(status_word(qkv.device).data_ptr()), _stream())
     if code == _UNSUPPORTED:
         return False
     if code != 0:
@@ -614,11 +615,11 @@ def wide_row_chunk_keys(blocks_per_chunk: int, context_bucket: int, window) -> i
 
 
 def prompt_attention(q, out, k_cache, v_cache, n_heads, n_kv_heads, head_dim, scale, window, keep_first,
-                     ctx, cache, table) -> bool:
+                     ctx, cache, table, chunked: bool = False, sinks=None, out_scale: float = 1.0) -> bool:
     """The tcgen05 attention for a step that holds portions of prompts only (no single decoded
     tokens ahead of them) over keys and values of one size, 64 or 128, with a window that may
-    keep the first tokens: plain softmax, no gate.  `q`: rows of n_heads * head_dim.  False:
-    not taken."""
+    keep the first tokens or (`chunked`) is the size of chunks, and with a sink per head in the
+    softmax (`sinks`) or none; no gate.  `q`: rows of n_heads * head_dim.  False: not taken."""
     host = getattr(ctx, "host", None)
     n_rep = n_heads // n_kv_heads
     if (not USE_TCGEN05_ATTENTION or host is None or q.dtype != torch.bfloat16 or head_dim not in (64, 128)
@@ -628,7 +629,7 @@ def prompt_attention(q, out, k_cache, v_cache, n_heads, n_kv_heads, head_dim, sc
         return False
     reqs = _Requests(ctx, table, 0, ctx.n_requests, host.max_new_tokens, host.context_bucket, ctx.n_tokens)
     return _attention_tcgen05(q, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, head_dim, scale, window, cache,
-                              keep_first=keep_first)
+                              keep_first=keep_first, chunked=chunked, sinks=sinks, out_scale=out_scale)
 
 
 SPLIT_ROWS = 16          # packed rows (new tokens x heads of a group) the split form takes

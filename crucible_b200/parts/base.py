@@ -19,7 +19,9 @@ position        `rotation() -> (cos, sin, rotary_dim) | None`, or
 mixer           `cache_need() -> CacheNeed | None`, `state_bytes() -> int`,
                 `forward(ctx, h, residual, binding)`: residual += mixer(h)
 feed-forward    `forward(ctx, h, residual)`: residual += ffn(h)
-arrangement     `norm_names`; `forward(ctx, x, binding)`: runs one layer on the residual x
+arrangement     `norm_names`; `forward(ctx, x, binding)`: runs one layer on the residual x;
+                one that remembers something of a request gives `own_state_bytes() -> int`
+                and finds it by `binding.own`
 embedding       `forward(ctx, token_ids) -> x`  fp32 [T, width]; `table` if a head may tie to it
 head            `forward(ctx, normed_rows) -> logits` fp32 [rows, vocab]; `tie(table)`
 
@@ -65,6 +67,8 @@ class CacheNeed:
     value_dim: Optional[int] = None   # size of a value, if it differs from a key's
     keep_first: int = 0            # with a window: this many first tokens stay visible
     values_are_keys: bool = False  # one row per token serves as key and as value: no value pages
+    chunked: bool = False          # the window is the size of chunks counted from position 0: a token
+                                   # reads the keys of its own chunk
 
 
 @dataclass(frozen=True)
@@ -72,12 +76,14 @@ class LayerBinding:
     """Where one run-order entry's mixer keeps what outlives a step: its cache
     group and the layer's slot inside that group's pages (group None: no paged
     cache), whether this run writes them (an entry that reads another layer's
-    cache does not), and its byte range inside each request's state slot."""
+    cache does not), its byte range inside each request's state slot, and the range
+    that belongs to the layer's arrangement (`own`)."""
     group: Optional[int] = None
     slot: int = 0
     write: bool = True
     state_offset: int = 0
     state_bytes: int = 0
+    own: Optional["LayerBinding"] = None
 
 
 class Part:

@@ -1,10 +1,11 @@
 """Block arrangements.  `pre_norm` is the only one the reference runs on the
 GPU (`model.py:262-264`, `engine/src/gpu_model.rs:518-520`):
 x = x + mixer(norm(x)); x = x + ffn(norm(x)).  `parallel` has one norm that both
-sublayers read: with n = norm(x), x = x + mixer(n) + ffn(n)."""
+sublayers read: with n = norm(x), x = x + mixer(n) + ffn(n).  `pre_norm_conv` is `pre_norm`
+with a short causal convolution on what each sublayer reads."""
 from __future__ import annotations
 
-from .base import ARRANGEMENTS, Arrangement
+from .base import ARRANGEMENTS, Arrangement, TensorDecl
 
 
 class PreNormBlock(Arrangement):
@@ -79,5 +80,62 @@ class ParallelBlock(Arrangement):
             self.feed_forward.forward(ctx, n, x)
 
 
+class PreNormConvBlock(PreNormBlock):
+    """x += mixer(c1(norm(x))); x += ffn(c2(norm(x))), c(h)_t = h_t + sum_j w_j h_(t - taps + 1 + j)
+    along a request's tokens, channel by channel (zeros before its start).  Norm, convolution and
+    sum are one launch, in 32 bits.  Option `taps` of the layer; tensors `mixer_conv` and
+    `feed_forward_conv` [width, taps] (the last column meets the current token).  The last
+    taps - 1 rows h of both sublayers are state of the layer's run."""
+
+    def __init__(self, spec, norms, mixer, feed_forward):
+        super().__init__(spec, norms, mixer, feed_forward)
+        self.taps = int(spec.option("taps", 4))
+        if not 1 <= self.taps <= 64:
+            raise ValueError(f"pre_norm_conv: 1 to 64 taps, got {self.taps}")
+        self.width = spec.mixer.width
+        self.tail_bytes = (4 * (self.taps - 1) * self.width + 15) // 16 * 16
+        self.conv = {}
+        self.dtype = None
+
+    @property
+    def sublayers(self):
+        return ("mixer", "feed_forward") if self.has_ffn else ("mixer",)
+
+    def tensors(self):
+        return [TensorDecl(f"{s}_conv", (self.width, self.taps), role="vector", init=("uniform", -0.5, 0.5))
+                for s in self.sublayers]
+
+    def bind(self, tensors, dtype, device):
+        self.dtype = dtype
+        # tap by tap, so that neighbouring columns lie side by side
+        self.conv = {s: tensors[f"{s}_conv"].t().contiguous() for s in self.sublayers}
+
+    def own_state_bytes(self) -> int:
+        return self.tail_bytes * len(self.sublayers)
+
+    def entry_norm(self):
+        return None          # the norm's rows go through the convolution: no product takes them as they are
+
+    def forward(self, ctx, x, binding):
+        announce = getattr(ctx, "announce_norm", None)
+        if announce is not None:
+            announce(None, None)
+        self.mixer.forward(ctx, self._read(ctx, x, binding, "mixer", 0), x, binding)
+        if not self.has_ffn:
+            return
+        h = self._read(ctx, x, binding, "feed_forward", self.tail_bytes)
+        self._announce(ctx, getattr(ctx, "norm_after_layer", None), x)
+        self.feed_forward.forward(ctx, h, x)
+
+    def _read(self, ctx, x, binding, sublayer, tail_off):
+        from ..ops import input_conv
+        norm = self.norms[f"{sublayer}_norm"]
+        out = ctx.scratch("norm.out", x.shape, self.dtype)
+        state = ctx.state(binding.own) if binding.own is not None else None
+        input_conv.norm_conv(x, norm.gain, norm.spec.eps, self.conv[sublayer], ctx, state, tail_off, out)
+        return out
+
+
 ARRANGEMENTS.register("pre_norm", PreNormBlock)
+ARRANGEMENTS.register("pre_norm_conv", PreNormConvBlock)
 ARRANGEMENTS.register("parallel", ParallelBlock)

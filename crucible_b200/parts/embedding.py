@@ -112,14 +112,17 @@ class HashedPositionEmbedding(Embedding):
 
 
 class LMHead(Head):
-    """logits = rows W^T; option `softcap` (a positive number c): logits <- c tanh(logits / c)."""
+    """logits = rows W^T; option `softcap` (a positive number c): logits <- c tanh(logits / c);
+    option `scale`: logits <- scale * (rows W^T) (before a cap; the model's final norm carries
+    the factor, see `DecoderModel.bind`)."""
 
-    def __init__(self, vocab_size: int, width: int, tied: bool, softcap=None):
+    def __init__(self, vocab_size: int, width: int, tied: bool, softcap=None, scale=None):
         self.vocab_size = vocab_size
         self.width = width
         self.tied = tied
         self.weight = None
         self.softcap = float(softcap) if softcap else None
+        self.scale = 1.0 if scale is None else float(scale)
         if self.softcap is not None and not self.softcap > 0:
             raise ValueError(f"the head's soft cap must be positive, got {softcap!r}")
 
@@ -145,4 +148,5 @@ class LMHead(Head):
 EMBEDDINGS.register("token", lambda spec, vocab, width: TokenEmbedding(vocab, width))
 EMBEDDINGS.register("token_normed_streams", NormedStreamsEmbedding)
 EMBEDDINGS.register("token_hashed_positions", HashedPositionEmbedding)
-HEADS.register("linear", lambda spec, vocab, width, tied: LMHead(vocab, width, tied, spec.option("softcap")))
+HEADS.register("linear", lambda spec, vocab, width, tied: LMHead(vocab, width, tied, spec.option("softcap"),
+                                                                spec.option("scale")))

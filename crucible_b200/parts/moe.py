@@ -13,7 +13,12 @@ which a token uses the `top` with the largest router logits z = h Wr^T (float32;
 index on ties), weighted by the softmax over those `top` logits alone; an optional shared
 expert of the same form runs for every token and is added.  Options: `router_bias` (the
 logits are h Wr^T + b, tensor `router.b`), `pair` = (limit, alpha, offset): the experts use
-the capped gated pair instead of silu(g) * u.
+the capped gated pair instead of silu(g) * u; `groups` = (count, keep): the experts form `count`
+equal groups of neighbours, a group's score is its best logit, and only the experts of the `keep`
+best groups can be chosen; `shared_gate` (tensor `shared.sg` [1, width]): the shared expert's result
+is multiplied by sigmoid(h Wsg^T), one number a token; `out_scale`: everything times this number.
+(The softmax over the chosen logits alone is the chosen experts' softmax over all experts divided
+by their sum.)
 """
 from __future__ import annotations
 
@@ -88,6 +93,7 @@ class MixtureOfExperts(FeedForward):
     SMALL_MAX_PAIRS = 256        # up to this many pairs the experts' weight rows are read by a warp each
     SORTED_MIN_PAIRS = 256       # from this many (token, expert) pairs on, a prompt step's experts
                                  # run as two grouped products over their rows side by side
+    MAX_EXPERTS = 256
 
     def __init__(self, spec: FeedForwardSpec):
         self.spec = spec
@@ -96,16 +102,36 @@ class MixtureOfExperts(FeedForward):
         self.ff = int(spec.intermediate)
         shared = spec.option("shared_intermediate")
         self.has_bias = bool(spec.option("router_bias", False))
+        self.shared_gate = bool(spec.option("shared_gate", False))
+        self.out_scale = float(spec.option("out_scale", 1.0))
+        groups = spec.option("groups")
+        self.groups = (int(groups[0]), int(groups[1])) if groups is not None else None
         pair = spec.option("pair")
         self.pair = tuple(float(v) for v in pair) if pair is not None else None
         if self.pair is not None and (len(self.pair) != 3 or not self.pair[0] > 0):
             raise ValueError("moe: pair is (limit > 0, alpha, offset)")
         if self.n <= 0 or not 0 < self.top <= self.n or self.ff <= 0:
             raise ValueError("moe: experts, top (at most experts) and the experts' ff must be positive")
-        if self.n > 256 or self.top > 32:
+        if self.n > self.MAX_EXPERTS or self.top > 32:
             raise ValueError("moe: up to 256 experts, of which a token uses up to 32")
-        self.shared = (SwiGLU(FeedForwardSpec(kind="swiglu", width=spec.width, intermediate=int(shared)))
-                       if shared else None)
+        if self.groups is not None:
+            count, keep = self.groups
+            if count <= 0 or self.n % count or not 0 < keep <= count or self.top > keep * (self.n // count):
+                raise ValueError("moe: groups = (count, keep): count divides the experts, keep is at most "
+                                 "count, and the kept groups hold at least `top` experts")
+        if shared and self.shared_gate and self.pair is not None:
+            raise ValueError("moe: a gated shared expert has no capped pair")
+        if shared and not self.shared_gate and self.out_scale != 1.0:
+            raise ValueError("moe: a shared expert without a gate takes no out_scale")
+        self.shared_ff = int(shared) if shared else 0
+        self.shared = (SwiGLU(FeedForwardSpec(kind="swiglu", width=spec.width, intermediate=self.shared_ff))
+                       if shared and not self.shared_gate else None)
+        self.shared_gate = self.shared_gate and self.shared_ff > 0
+        # A gated shared expert as slices of an expert's size (the last one padded with zeros) that
+        # every token chooses: a few rows then take no launches of their own for it.
+        self.slices = -(-self.shared_ff // self.ff) if self.shared_gate else 0
+        if self.slices > 32 or self.n + self.slices > self.MAX_EXPERTS:
+            self.slices = 0
 
     def tensors(self):
         d, f = self.spec.width, self.ff
@@ -117,29 +143,57 @@ class MixtureOfExperts(FeedForward):
                     TensorDecl(f"e{e}.down", (d, f))]
         if self.shared is not None:
             out += [TensorDecl(f"shared.{t.name}", t.shape, t.role) for t in self.shared.tensors()]
+        elif self.shared_gate:
+            fs = self.shared_ff
+            out += [TensorDecl("shared.gate", (fs, d)), TensorDecl("shared.up", (fs, d)),
+                    TensorDecl("shared.down", (d, fs)), TensorDecl("shared.sg", (1, d))]
         return out
 
     def bind(self, tensors, dtype, device):
         self.dtype = dtype
-        self.router = tensors["router"]
+        d, f = self.spec.width, self.ff
+        # the router's rows and, behind them, the row of the shared expert's gate: one product
+        self.router = (torch.cat([tensors["router"], tensors["shared.sg"]], 0).contiguous()
+                       if self.shared_gate else tensors["router"])
         self.router_bias = tensors.get("router.b") if self.has_bias else None
-        self.gate_up = torch.stack([torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], 0)
-                                    for e in range(self.n)], 0).contiguous()          # [E, 2F, d]
-        self.down = torch.stack([tensors[f"e{e}.down"] for e in range(self.n)], 0).contiguous()   # [E, d, F]
+        gate_up = [torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], 0) for e in range(self.n)]
+        down = [tensors[f"e{e}.down"] for e in range(self.n)]
+        for s in range(self.slices):
+            lo, hi = s * f, min((s + 1) * f, self.shared_ff)
+            gu, dn = torch.zeros((2 * f, d), dtype=dtype, device=device), torch.zeros((d, f), dtype=dtype, device=device)
+            gu[:hi - lo], gu[f:f + hi - lo] = tensors["shared.gate"][lo:hi], tensors["shared.up"][lo:hi]
+            dn[:, :hi - lo] = tensors["shared.down"][:, lo:hi]
+            gate_up.append(gu)
+            down.append(dn)
+        self.gate_up = torch.stack(gate_up, 0).contiguous()          # [E + slices, 2F, d]
+        self.down = torch.stack(down, 0).contiguous()                # [E + slices, d, F]
         ops.declare_weights(self.router, self.gate_up, self.down)
-        self.count = torch.zeros(self.n, dtype=torch.int32, device=device)     # zero between steps
+        # the shared expert as dense products, for steps of many rows
+        self.dense = []
+        if self.shared_gate:
+            if self.slices:
+                self.dense = [(self.gate_up[self.n + s], self.down[self.n + s]) for s in range(self.slices)]
+            else:
+                self.dense = [(torch.cat([tensors["shared.gate"], tensors["shared.up"]], 0).contiguous(),
+                               tensors["shared.down"])]
+                ops.declare_weights(*self.dense[0])
+        self.count = torch.zeros(self.n + self.slices, dtype=torch.int32, device=device)     # zero between steps
         if self.shared is not None:
             self.shared.bind({k[len("shared."):]: v for k, v in tensors.items() if k.startswith("shared.")},
                              dtype, device)
 
     def forward(self, ctx, h, residual):
-        t, d, top, n, f = h.shape[0], self.spec.width, self.top, self.n, self.ff
-        logits = ctx.scratch("moe.logits", (t, n), torch.float32)
+        t, d, f = h.shape[0], self.spec.width, self.ff
+        logits = ctx.scratch("moe.logits", (t, self.router.shape[0]), torch.float32)
         ops.linear(h, self.router, logits)
         # many rows of a prompt: the experts' rows side by side and two grouped products on the
-        # tensor cores, by the plan on the device (tiles of 128 rows)
-        grouped = (self.dtype == torch.bfloat16 and t * top >= self.SORTED_MIN_PAIRS
+        # tensor cores, by the plan on the device (tiles of 128 rows); a gated shared expert then
+        # runs as dense products of its own
+        grouped = (self.dtype == torch.bfloat16 and t * self.top >= self.SORTED_MIN_PAIRS
                    and ctx.host.max_new_tokens > 1 and d % 8 == 0 and f % 8 == 0)
+        riding = 0 if grouped else self.slices
+        apart = self.shared_gate and not riding
+        n, top = self.n + riding, self.top + riding              # experts of the plan, pairs of a token
         tile_rows = kernels.GROUPED_TILE_ROWS if grouped else 0
         tiles = kernels.max_tiles(t, top, n, tile_rows)
         idx = ctx.scratch("moe.idx", (t * top,), torch.int32)
@@ -147,30 +201,39 @@ class MixtureOfExperts(FeedForward):
         order = ctx.scratch("moe.order", (t * top,), torch.int32)
         weight = ctx.scratch("moe.weight", (t * top,), torch.float32)
         plan = ctx.scratch("moe.plan", (kernels.plan_ints(n, tiles),), torch.int32)
-        kernels.route(logits, top, idx, weight, place, self.count, plan, tiles, order, bias=self.router_bias,
-                      rows=tile_rows)
+        gate = ctx.scratch("moe.shared_gate", (t,), torch.float32) if apart else None
+        kernels.route(logits, self.top, idx, weight, place, self.count, plan, tiles, order, bias=self.router_bias,
+                      rows=tile_rows, n_experts=self.n, groups=self.groups, n_shared=riding,
+                      gate_col=self.n if self.shared_gate else -1, scale=self.out_scale, gate_out=gate)
         act = ctx.scratch("moe.act", (t * top, f), self.dtype)
-        pair_out = ctx.scratch("moe.pair_out", (t * top, d), torch.float32)
+        by_plan = None
         if grouped:
             rows = ctx.scratch("moe.rows", (t * top, d), self.dtype)
             kernels.gather(h, order, top, rows)
-            down = ctx.scratch("moe.down", (t * top, d), torch.float32)
+            pair_out = ctx.scratch("moe.down", (t * top, d), torch.float32)
             if not (kernels.grouped_linear(rows, self.gate_up, act, plan, n, tiles, True, pair=self.pair)
-                    and kernels.grouped_linear(act, self.down, down, plan, n, tiles, False)):
+                    and kernels.grouped_linear(act, self.down, pair_out, plan, n, tiles, False)):
                 raise RuntimeError("moe: the grouped product refused sizes its rule allows")
-            kernels.scatter(down, order, weight, pair_out)
-        elif (self.dtype == torch.bfloat16 and t * top <= self.SMALL_MAX_PAIRS
-              and kernels.expert_rows_small(True, h, self.gate_up, f, plan, n, tiles, order, top, weight, act,
-                                            pair=self.pair)):
-            # few rows (decoded tokens): the weights are what moves; a warp per weight row
-            if not kernels.expert_rows_small(False, act, self.down, d, plan, n, tiles, order, top, weight,
-                                             pair_out):
-                kernels.expert_tiles(False, act, self.down, d, plan, n, tiles, order, top, weight, pair_out)
+            by_plan = (plan, idx, place, weight)
         else:
-            kernels.expert_tiles(True, h, self.gate_up, f, plan, n, tiles, order, top, weight, act,
-                                 pair=self.pair)
-            kernels.expert_tiles(False, act, self.down, d, plan, n, tiles, order, top, weight, pair_out)
-        kernels.combine(pair_out, top, residual)
+            pair_out = ctx.scratch("moe.pair_out", (t * top, d), torch.float32)
+            # few rows (decoded tokens): the weights are what moves; a warp per weight row
+            small = self.dtype == torch.bfloat16 and t * top <= self.SMALL_MAX_PAIRS
+            if not (small and kernels.expert_rows_small(True, h, self.gate_up, f, plan, n, tiles, order, top, weight,
+                                                        act, pair=self.pair)):
+                kernels.expert_tiles(True, h, self.gate_up, f, plan, n, tiles, order, top, weight, act,
+                                     pair=self.pair)
+            if not (small and kernels.expert_rows_small(False, act, self.down, d, plan, n, tiles, order, top, weight,
+                                                        pair_out)):
+                kernels.expert_tiles(False, act, self.down, d, plan, n, tiles, order, top, weight, pair_out)
+        shared_out = None
+        if apart:
+            shared_out = ctx.scratch("moe.shared_out", (t, d), torch.float32)
+            for i, (gate_up, down) in enumerate(self.dense):
+                shared_act = ctx.scratch("moe.shared_act", (t, down.shape[1]), self.dtype)
+                ops.linear_swiglu(h, gate_up, shared_act, ctx)
+                ops.linear(shared_act, down, shared_out, accumulate=i > 0)
+        kernels.combine(pair_out, top, residual, by_plan=by_plan, shared=shared_out, gate=gate)
         if self.shared is not None:
             self.shared.forward(ctx, h, residual)
 

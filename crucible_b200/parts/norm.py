@@ -28,6 +28,10 @@ class RMSNorm(Norm):
         self.gain = tensors["gain"]
         self.dtype = dtype
 
+    def scale_gain(self, factor: float) -> None:
+        """Every result times `factor` from here on (after `bind`)."""
+        self.gain = (self.gain * factor).contiguous()
+
     supports_lazy = True
     supports_ahead = True      # the product that writes the rows last may leave this norm's input
 
@@ -63,5 +67,17 @@ class OffsetRMSNorm(RMSNorm):
         self.gain = (tensors["gain"].to(torch.float32) + 1.0).contiguous()
 
 
+class OneNumberRMSNorm(RMSNorm):
+    """RMSNorm with ONE stored number as the gain of every coordinate (a tensor of shape [])."""
+
+    def tensors(self):
+        return [TensorDecl("gain", (), role="vector", init=("normal", 1.0, 0.1))]
+
+    def bind(self, tensors, dtype, device):
+        super().bind(tensors, dtype, device)
+        self.gain = tensors["gain"].to(torch.float32).reshape(1).expand(self.spec.width).contiguous()
+
+
 NORMS.register("rmsnorm", RMSNorm)
+NORMS.register("rmsnorm_one_number", OneNumberRMSNorm)
 NORMS.register("rmsnorm_offset", OffsetRMSNorm)

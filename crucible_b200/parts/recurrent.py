@@ -10,6 +10,13 @@ beta = sigmoid(h Wb^T) and g = exp(-exp(A_log) * softplus(h Wa^T + dt_bias)):
     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
 o / rms(o) * norm [E] * silu(h Wg^T) goes through Wo.  Head i uses q/k head i // (H / G).
 
+`channel_delta` (the delta rule with a decay per key channel): q, k, v as in `gated_delta`
+(option `conv_taps`); beta = sigmoid(h Wb^T) per head; per head and key channel
+g = exp(-exp(A_log) * softplus((h Wa1^T) Wa2^T + dt_bias)) [H, D].  Per head:
+    S <- diag(g) S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q.
+o / rms(o) * norm [E] * sigmoid((h Wg1^T) Wg2^T) goes through Wo, times the option `out_scale`.
+The two low ranks are whatever the checkpoint gives them.
+
 `mlstm` (the matrix memory of the xLSTM): q = h Wq^T * D^-1/2, k [H, D], v [H, E];
 log gates i = cap * tanh((h Wi^T + bi) / cap), f = logsigmoid(cap * tanh((h Wf^T + bf) / cap));
 with m (from 0):  m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;
@@ -107,6 +114,82 @@ class GatedDeltaRule(BranchMixer):
                               0, o, H, G, D, E)
         kernels.head_norm_gate(o, self.gain, False, proj[:, C:C + H * E], act, kernels.GATE_SILU, H, E,
                                self.eps, out_scale)
+
+
+class ChannelDeltaRule(BranchMixer):
+    def __init__(self, spec: MixerSpec):
+        s = self.spec = spec
+        self.H, self.G, self.D = s.n_heads, s.n_kv_heads, s.head_dim
+        self.E = int(s.option("value_dim", s.head_dim))
+        self.taps = int(s.option("conv_taps", 4))
+        self.rank = int(s.option("rank", 16))          # of the random-weights mode
+        self.eps = float(s.option("norm_eps", 1e-6))
+        self.out_scale = float(s.option("out_scale", 1.0))
+        if self.H <= 0 or self.G <= 0 or self.H % self.G or self.D <= 0 or self.E <= 0:
+            raise ValueError("channel_delta: heads must be a multiple of kv_heads; sizes positive")
+        if self.D > 256 or not 1 <= self.taps <= 64:
+            raise ValueError("channel_delta: key size up to 256, 1 to 64 taps")
+        self.C = 2 * self.G * self.D + self.H * self.E          # channels under the convolution
+        self.s_bytes = _round16(4 * self.H * self.D * self.E)
+        self.tail_bytes = 4 * (self.taps - 1) * self.C
+
+    def tensors(self):
+        d, H, G, D, E, r = self.spec.width, self.H, self.G, self.D, self.E, self.rank
+        conv = ("uniform", -0.5, 0.5)
+        return [TensorDecl("q", (G * D, d)), TensorDecl("k", (G * D, d)), TensorDecl("v", (H * E, d)),
+                TensorDecl("q.conv", (G * D, self.taps), role="vector", init=conv),
+                TensorDecl("k.conv", (G * D, self.taps), role="vector", init=conv),
+                TensorDecl("v.conv", (H * E, self.taps), role="vector", init=conv),
+                TensorDecl("b", (H, d)),
+                TensorDecl("A_log", (H,), role="vector", init=("uniform", -1.0, 1.0)),
+                TensorDecl("a1", (r, d), free_dims=(0,)), TensorDecl("a2", (H * D, r), free_dims=(1,)),
+                TensorDecl("dt_bias", (H * D,), role="vector", init=("uniform", -4.0, 0.0)),
+                TensorDecl("norm", (E,), role="vector"),
+                TensorDecl("g1", (r, d), free_dims=(0,)), TensorDecl("g2", (H * E, r), free_dims=(1,)),
+                TensorDecl("o", (d, H * E))]
+
+    def bind(self, tensors, dtype, device):
+        H, D, E, d = self.H, self.D, self.E, self.spec.width
+        for name in ("a", "g"):
+            if tensors[f"{name}1"].shape[0] != tensors[f"{name}2"].shape[1]:
+                raise ValueError(f"channel_delta: {name}1 and {name}2 disagree on their rank")
+        ra, rg = int(tensors["a1"].shape[0]), int(tensors["g1"].shape[0])
+        pa, pg = -(-ra // 8) * 8, -(-rg // 8) * 8
+        zeros = lambda rows, cols: torch.zeros((rows, cols), dtype=dtype, device=device)
+        # the joint projection: [q | k | v | spare | a1 | spare | g1 | spare], the two low ranks side by
+        # side from a column that is a multiple of 8 on (rows of whole 16-byte pieces) ...
+        self.low_at, self.low = -(-self.C // 8) * 8, pa + pg
+        self.w_in = torch.cat([tensors["q"], tensors["k"], tensors["v"], zeros(self.low_at - self.C, d),
+                               tensors["a1"], zeros(pa - ra, d), tensors["g1"], zeros(pg - rg, d)], 0).contiguous()
+        # ... and one product out of both: [a2 | 0] over [0 | g2]
+        self.w_low = zeros(H * (D + E), self.low)
+        self.w_low[:H * D, :ra] = tensors["a2"]
+        self.w_low[H * D:, pa:pa + rg] = tensors["g2"]
+        self.w_gates = tensors["b"]
+        self.w_out = tensors["o"]
+        self.conv_w = torch.cat([tensors["q.conv"], tensors["k.conv"], tensors["v.conv"]], 0).t().contiguous()
+        self.a_log, self.dt_bias, self.gain = tensors["A_log"], tensors["dt_bias"], tensors["norm"]
+        self.dtype = dtype
+        self._declare()
+        ops.declare_weights(self.w_low)
+
+    def state_bytes(self) -> int:
+        return self.s_bytes + self.tail_bytes
+
+    def run_branch(self, ctx, proj, gates, act, out_scale, binding):
+        t, H, G, D, E, C = proj.shape[0], self.H, self.G, self.D, self.E, self.C
+        state = ctx.state(binding)
+        logits = ctx.scratch("channel.logits", (t, H * (D + E)), torch.float32)      # [decay rates | output gate]
+        ops.linear(proj[:, self.low_at:self.low_at + self.low], self.w_low, logits)
+        qkv = ctx.scratch("channel.qkv", (t, C + H * D), torch.float32)
+        beta = ctx.scratch("channel.beta", (t, H), torch.float32)
+        o = ctx.scratch("channel.o", (t, H * E), torch.float32)
+        kernels.channel_delta_prepare(proj, self.conv_w, logits, gates, self.a_log, self.dt_bias, ctx, state,
+                                      self.s_bytes, qkv, beta, H, G, D, E)
+        kernels.matrix_memory(kernels.CHANNEL, qkv, 0, G * D, 2 * G * D, None, beta, ctx, state, 0, 0, 0, o,
+                              H, G, D, E, w_off=C)
+        kernels.head_norm_gate(o, self.gain, False, logits[:, H * D:], act, kernels.GATE_SIGMOID, H, E, self.eps,
+                               out_scale * self.out_scale)
 
 
 class MLSTM(BranchMixer):
@@ -345,6 +428,7 @@ class Retention(BranchMixer):
 
 
 MIXERS.register("gated_delta", GatedDeltaRule)
+MIXERS.register("channel_delta", ChannelDeltaRule)
 MIXERS.register("retention", Retention)
 MIXERS.register("wkv", WKVMixer)
 MIXERS.register("mamba2", StateSpaceMixer)

@@ -17,8 +17,10 @@ head, `g` [H, width]; false: none), qk_norm_eps (default None; a number: every q
 divided by its root mean square over D, that eps under the root, and multiplied by the weight
 `q.norm` / `k.norm` of size D that all heads share, before the rotation), qk_norm_whole
 (default false; true: the root mean square is taken over the whole projection, all H * D
-features of q at once and all G * D of k, and the weights have those sizes).  `window` None
-means every earlier key.
+features of q at once and all G * D of k, and the weights have those sizes), chunked (default
+false; true: `window` is the size of chunks counted from position 0 and a row sees the keys of its
+own chunk up to itself), out_scale (the result times this, default 1).  `window` None means every
+earlier key.
 The position encoding says which features pair (`split_halves`: i with i + R/2, else
 neighbours).
 """
@@ -34,6 +36,10 @@ from .branch import BranchMixer
 
 class SinkWindowAttention(BranchMixer):
     def __init__(self, spec: MixerSpec):
+        self.chunked = bool(spec.option("chunked", False))
+        self.out_scale = float(spec.option("out_scale", 1.0))
+        if self.chunked and (spec.window is None or spec.option("keep_first", 0)):
+            raise ValueError("chunked attention: the window is the chunks' size and no first tokens are kept")
         if spec.n_heads <= 0 or spec.n_kv_heads <= 0 or spec.head_dim <= 0:
             raise ValueError("attention needs positive n_heads, n_kv_heads and head_dim")
         if spec.n_heads % spec.n_kv_heads != 0:
@@ -98,7 +104,7 @@ class SinkWindowAttention(BranchMixer):
         s = self.spec
         return CacheNeed(kv_heads=s.n_kv_heads, head_dim=s.head_dim, window=s.window,
                          value_dim=self.value_dim if self.value_dim != s.head_dim else None,
-                         keep_first=self.keep_first if s.window is not None else 0)
+                         keep_first=self.keep_first if s.window is not None else 0, chunked=self.chunked)
 
     def run_branch(self, ctx, proj, gates, act, out_scale, binding):
         s = self.spec
@@ -121,7 +127,8 @@ class SinkWindowAttention(BranchMixer):
                 if self.has_gate else None)
         kernels.attention(proj[:, :q_width], gate, act, self.sinks, s.n_heads, s.n_kv_heads,
                           s.head_dim, self.value_dim, s.softmax_scale, s.window, self.keep_first,
-                          out_scale, ctx, cache, binding, gate_per_head=per_head)
+                          out_scale * self.out_scale, ctx, cache, binding, gate_per_head=per_head,
+                          chunked=self.chunked)
 
 
 MIXERS.register("sink_attention", SinkWindowAttention)
