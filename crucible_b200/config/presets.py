@@ -160,3 +160,31 @@ def sebalorn(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, voca
 
 SHAPES["sebalorn-w1024"] = sebalorn(*COMPARISON_SIZES["w1024"])
 SHAPES["sebalorn-w2048"] = sebalorn(*COMPARISON_SIZES["w2048"])
+
+
+def ramalix(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, vocab: int,
+            layers: int = 4, experts: int = 8, top: int = 2, chunk: int = 1024, passes: int = 1) -> dict:
+    """A Ramalix config.json of a real model's proportions: `layers` layers that take turns as
+    chunked attention with a sink, the delta rule with a decay per key channel, differential
+    attention (its maps' keys half a value wide), the delta rule; every mixer `heads * head_dim`
+    wide; `experts` experts of half the dense width in four groups of which two take part, a token
+    uses `top` of them and a gated shared expert of the same size.  Layers 1 and 2 form the
+    repeated run, `passes` times (1: every layer runs once)."""
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2}}
+    chunked = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+               "rot": {"base": 10000.0, "dims": head_dim // 2}, "mask": {"size": chunk}}
+    delta = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "conv": 4}
+    differential = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim // 2, "vdim": head_dim, "diff": 0.4,
+                    "scale": (head_dim // 2) ** -0.5, "q_temp": {"coef": 0.1, "every": 8192}}
+    cycle = [("attention_2", chunked), ("channel_delta", delta), ("attention", differential), ("channel_delta", delta)]
+    out = {"architecture": "Ramalix", "vocab": vocab, "width": width, "norm": {"eps": 1e-5}, "canon": {"taps": 4},
+           "residual_mult": 0.7, "logit_scale": 1.0,
+           "layers": [{"type": cycle[i % 4][0], "mixer": dict(cycle[i % 4][1]), "mlp": moe} for i in range(layers)]}
+    if layers >= 3:
+        out["loop"] = {"start": 1, "stop": 3, "times": passes}
+    return out
+
+
+SHAPES["ramalix-w1024"] = ramalix(*COMPARISON_SIZES["w1024"])
+SHAPES["ramalix-w2048"] = ramalix(*COMPARISON_SIZES["w2048"])

@@ -36,123 +36,171 @@ __device__ __forceinline__ float gated_f(float g, float u, const GateRule& p) {
     return g / (1.0f + expf(-p.alpha * g)) * (u + p.offset);
 }
 
-__global__ void moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias,
-                                 int n_tokens, int stride, int E, int top,
-                                 int* __restrict__ idx, float* __restrict__ weight,
-                                 int* __restrict__ place, int* __restrict__ count, int groups, int keep,
-                                 int n_shared, int gate_col, float scale, float* __restrict__ gate_out) {
+constexpr int ROUTE_WARPS = 8;        // of a routing block ...
+constexpr int ROUTE_TOKENS = 4;       // ... each of which takes up to this many tokens
+constexpr int MAX_TOTAL = 32 * MAX_PER_LANE + 32;      // routed experts and a shared expert's slices
+
+// A pair's place among its expert's pairs: a counter per expert in shared memory, then one addition
+// per block and expert to the global counter.
+__global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(
+    const float* __restrict__ logits, const float* __restrict__ bias, int n_tokens, int stride, int E, int top,
+    int* __restrict__ idx, float* __restrict__ weight, int* __restrict__ place, int* __restrict__ count,
+    int groups, int keep, int n_shared, int gate_col, float scale, float* __restrict__ gate_out, int per_warp) {
     cb_pdl_trigger();
     cb_pdl_wait();
-    const int t = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    if (t >= n_tokens) return;
-    const int lane = threadIdx.x & 31;
-    float v[MAX_PER_LANE];
+    __shared__ float all[ROUTE_WARPS][32 * MAX_PER_LANE], best_of[ROUTE_WARPS][32 * MAX_PER_LANE];
+    __shared__ int block_count[32 * MAX_PER_LANE], block_base[32 * MAX_PER_LANE];
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int e = threadIdx.x; e < E; e += blockDim.x) block_count[e] = 0;
+    __syncthreads();
+    int chosen[ROUTE_TOKENS], in_block[ROUTE_TOKENS];
+    const int t0 = (blockIdx.x * ROUTE_WARPS + warp) * per_warp;
 #pragma unroll
-    for (int i = 0; i < MAX_PER_LANE; ++i) {
-        const int e = lane + 32 * i;
-        v[i] = e < E ? logits[(size_t)t * stride + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
-    }
-    if (keep < groups) {
-        // only the experts of the `keep` groups with the largest best logit (the lower group on
-        // equal ones) stay
-        __shared__ float all[4][32 * MAX_PER_LANE], best_of[4][32 * MAX_PER_LANE];
-        const int warp = threadIdx.x >> 5, size = E / groups;
-#pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i)
-            if (lane + 32 * i < E) all[warp][lane + 32 * i] = v[i];
-        __syncwarp();
-        for (int g = lane; g < groups; g += 32) {
-            float m = -INFINITY;
-            for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, all[warp][e]);
-            best_of[warp][g] = m;
-        }
-        __syncwarp();
+    for (int k = 0; k < ROUTE_TOKENS; ++k) {
+        const int t = t0 + k;
+        chosen[k] = -1;
+        if (k >= per_warp || t >= n_tokens) continue;
+        float v[MAX_PER_LANE];
 #pragma unroll
         for (int i = 0; i < MAX_PER_LANE; ++i) {
             const int e = lane + 32 * i;
-            if (e >= E) continue;
-            const int mine_g = e / size;
-            const float m = best_of[warp][mine_g];
-            int ahead = 0;
-            for (int g = 0; g < groups; ++g) ahead += best_of[warp][g] > m || (best_of[warp][g] == m && g < mine_g);
-            if (ahead >= keep) v[i] = -INFINITY;
+            v[i] = e < E ? logits[(size_t)t * stride + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
         }
-    }
-    float first = 0.f, total = 0.f, mine = 0.f;
-    int mine_e = 0;
-    for (int j = 0; j < top; ++j) {
-        float best = -INFINITY;
-        int best_e = 0x7fffffff;
+        if (keep < groups) {
+            // only the experts of the `keep` groups with the largest best logit (the lower group on
+            // equal ones) stay
+            const int size = E / groups;
+            __syncwarp();
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i) {
-            const int e = lane + 32 * i;
-            if (e < E && (v[i] > best || (v[i] == best && e < best_e))) { best = v[i]; best_e = e; }
-        }
+            for (int i = 0; i < MAX_PER_LANE; ++i)
+                if (lane + 32 * i < E) all[warp][lane + 32 * i] = v[i];
+            __syncwarp();
+            for (int g = lane; g < groups; g += 32) {
+                float m = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, all[warp][e]);
+                best_of[warp][g] = m;
+            }
+            __syncwarp();
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ob = __shfl_xor_sync(0xffffffffu, best, o);
-            const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
-            if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
+            for (int i = 0; i < MAX_PER_LANE; ++i) {
+                const int e = lane + 32 * i;
+                if (e >= E) continue;
+                const int mine_g = e / size;
+                const float m = best_of[warp][mine_g];
+                int ahead = 0;
+                for (int g = 0; g < groups; ++g)
+                    ahead += best_of[warp][g] > m || (best_of[warp][g] == m && g < mine_g);
+                if (ahead >= keep) v[i] = -INFINITY;
+            }
         }
-        if (best_e == 0x7fffffff) best_e = j < E ? j : 0;      // nothing comparable left (NaN logits)
+        float first = 0.f, total = 0.f, mine = 0.f;
+        int mine_e = 0;
+        for (int j = 0; j < top; ++j) {
+            float best = -INFINITY;
+            int best_e = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < MAX_PER_LANE; ++i)
-            if (lane + 32 * i == best_e) v[i] = -INFINITY;
-        if (j == 0) first = best;
-        const float p = expf(best - first);
-        total += p;
-        if (lane == j) { mine = p; mine_e = best_e; }
-    }
-    const size_t at = (size_t)t * (top + n_shared);
-    if (lane < top) {
-        idx[at + lane] = mine_e;
-        weight[at + lane] = mine / total * scale;
-        place[at + lane] = atomicAdd(&count[mine_e], 1);
-    }
-    if (gate_col >= 0) {
-        const float gate = scale / (1.0f + expf(-logits[(size_t)t * stride + gate_col]));
-        // the shared expert's slices: every token's, so its place among their pairs is its own number
-        for (int s = lane; s < n_shared; s += 32) {
-            idx[at + top + s] = E + s;
-            weight[at + top + s] = gate;
-            place[at + top + s] = t;
-            if (t == 0) count[E + s] = n_tokens;
+            for (int i = 0; i < MAX_PER_LANE; ++i) {
+                const int e = lane + 32 * i;
+                if (e < E && (v[i] > best || (v[i] == best && e < best_e))) { best = v[i]; best_e = e; }
+            }
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) {
+                const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+                const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+                if (ob > best || (ob == best && oe < best_e)) { best = ob; best_e = oe; }
+            }
+            if (best_e == 0x7fffffff) best_e = j < E ? j : 0;      // nothing comparable left (NaN logits)
+#pragma unroll
+            for (int i = 0; i < MAX_PER_LANE; ++i)
+                if (lane + 32 * i == best_e) v[i] = -INFINITY;
+            if (j == 0) first = best;
+            const float p = expf(best - first);
+            total += p;
+            if (lane == j) { mine = p; mine_e = best_e; }
         }
-        if (gate_out != nullptr && lane == 0) gate_out[t] = gate;
+        const size_t at = (size_t)t * (top + n_shared);
+        if (lane < top) {
+            idx[at + lane] = mine_e;
+            weight[at + lane] = mine / total * scale;
+            chosen[k] = mine_e;
+            in_block[k] = atomicAdd(&block_count[mine_e], 1);
+        }
+        if (gate_col >= 0) {
+            const float gate = scale / (1.0f + expf(-logits[(size_t)t * stride + gate_col]));
+            // the shared expert's slices: every token's, so its place among their pairs is its own number
+            for (int s = lane; s < n_shared; s += 32) {
+                idx[at + top + s] = E + s;
+                weight[at + top + s] = gate;
+                place[at + top + s] = t;
+                if (t == 0) count[E + s] = n_tokens;
+            }
+            if (gate_out != nullptr && lane == 0) gate_out[t] = gate;
+        }
     }
+    __syncthreads();
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+        const int n = block_count[e];
+        block_base[e] = n > 0 ? atomicAdd(&count[e], n) : 0;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int k = 0; k < ROUTE_TOKENS; ++k)
+        if (chosen[k] >= 0)
+            place[(size_t)(t0 + k) * (top + n_shared) + lane] = block_base[chosen[k]] + in_block[k];
 }
 
 // (tile_rows_: rows of a tile: TM for the kernels of this file, 128 for the tensor cores' grouped product)
 // plan: [0] number of tiles, [1 .. E+1] each expert's start in the sorted order, then
 // max_tiles each of (expert, start, rows).
-__global__ void moe_plan_kernel(int* __restrict__ count, int E, int n_pairs, const int* __restrict__ idx,
-                                const int* __restrict__ place, int* __restrict__ plan, int max_tiles,
-                                int* __restrict__ sorted_pair, int tile_rows_) {
+__global__ void __launch_bounds__(1024) moe_plan_kernel(int* __restrict__ count, int E, int n_pairs,
+                                                        const int* __restrict__ idx,
+                                                        const int* __restrict__ place, int* __restrict__ plan,
+                                                        int max_tiles, int* __restrict__ sorted_pair,
+                                                        int tile_rows_) {
     cb_pdl_trigger();
     cb_pdl_wait();
-    int* offsets = plan + 1;
+    __shared__ int start[MAX_TOTAL + 1], first_tile[MAX_TOTAL + 1];
     int* tile_expert = plan + 2 + E;
     int* tile_start = tile_expert + max_tiles;
     int* tile_rows = tile_start + max_tiles;
-    if (threadIdx.x == 0) {
-        int at = 0, tiles = 0;
-        for (int e = 0; e < E; ++e) {
-            offsets[e] = at;
-            const int n = count[e];
-            for (int r = 0; r < n && tiles < max_tiles; r += tile_rows_, ++tiles) {
-                tile_expert[tiles] = e;
-                tile_start[tiles] = at + r;
-                tile_rows[tiles] = min(tile_rows_, n - r);
+    if (threadIdx.x < 32) {
+        // running sums of the experts' pairs and tiles, 32 experts at a time
+        const int lane = threadIdx.x;
+        int pairs = 0, tiles = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int n = e0 + lane < E ? count[e0 + lane] : 0;
+            int a = n, b = (n + tile_rows_ - 1) / tile_rows_;
+            const int my_tiles = b;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const int ua = __shfl_up_sync(0xffffffffu, a, o), ub = __shfl_up_sync(0xffffffffu, b, o);
+                if (lane >= o) { a += ua; b += ub; }
             }
-            at += n;
+            if (e0 + lane < E) {
+                start[e0 + lane] = pairs + a - n;
+                first_tile[e0 + lane] = tiles + b - my_tiles;
+            }
+            pairs += __shfl_sync(0xffffffffu, a, 31);
+            tiles += __shfl_sync(0xffffffffu, b, 31);
         }
-        offsets[E] = at;
-        plan[0] = tiles;
+        if (lane == 0) {
+            start[E] = pairs;
+            first_tile[E] = tiles;
+            plan[0] = min(tiles, max_tiles);
+        }
     }
     __syncthreads();
-    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) sorted_pair[offsets[idx[p]] + place[p]] = p;
-    __syncthreads();
-    for (int e = threadIdx.x; e < E; e += blockDim.x) count[e] = 0;      // ready for the next step
+    for (int e = threadIdx.x; e <= E; e += blockDim.x) plan[1 + e] = start[e];
+    for (int e = threadIdx.x; e < E; e += blockDim.x) {
+        const int n = start[e + 1] - start[e];
+        for (int r = 0, tile = first_tile[e]; r < n && tile < max_tiles; r += tile_rows_, ++tile) {
+            tile_expert[tile] = e;
+            tile_start[tile] = start[e] + r;
+            tile_rows[tile] = min(tile_rows_, n - r);
+        }
+        count[e] = 0;                              // ready for the next step
+    }
+    for (int p = threadIdx.x; p < n_pairs; p += blockDim.x) sorted_pair[start[idx[p]] + place[p]] = p;
 }
 
 // GATED: rows are h[token of the pair], W = [gate rows; up rows] of the tile's expert,
@@ -412,9 +460,12 @@ CB_EXPORT int cb_moe_route(const float* logits, int stride, const float* bias, i
         (n_shared > 0 && gate_col < 0) || gate_col >= stride)
         return CB_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-    cb_launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, s, logits, bias, n_tokens, stride, E, top,
-              idx, weight, place, count, groups, keep, n_shared, gate_col, scale, gate_out);
-    cb_launch(moe_plan_kernel, dim3(1), dim3(256), 0, s, count, E + n_shared, n_tokens * (top + n_shared),
+    if (E + n_shared > MAX_TOTAL) return CB_ERR_UNSUPPORTED;
+    const int per_warp = n_tokens >= 1024 ? ROUTE_TOKENS : 1, per_block = ROUTE_WARPS * per_warp;
+    cb_launch(moe_route_kernel, dim3((n_tokens + per_block - 1) / per_block), dim3(32 * ROUTE_WARPS), 0, s, logits,
+              bias, n_tokens, stride, E, top, idx, weight, place, count, groups, keep, n_shared, gate_col, scale,
+              gate_out, per_warp);
+    cb_launch(moe_plan_kernel, dim3(1), dim3(n_tokens * (top + n_shared) > 256 ? 1024 : 256), 0, s, count, E + n_shared, n_tokens * (top + n_shared),
               (const int*)idx, (const int*)place, plan, max_tiles, sorted_pair, tile_rows > 0 ? tile_rows : TM);
     return cb_last_error();
 }
@@ -445,8 +496,9 @@ CB_EXPORT int cb_moe_rows_small(int gated, const void* a, int a_stride, const vo
     if (max_tiles <= 0) return 0;
     const GateRule rule = {limit, alpha, offset};
     if (K % 8 || a_stride % 8 || ((uintptr_t)a & 15) || ((uintptr_t)w & 15)) return CB_ERR_UNSUPPORTED;
-    // enough blocks to keep the memory busy: about four to an SM over all tiles
-    int chunks = (4 * 148 + max_tiles - 1) / max_tiles;
+    // enough blocks to keep the memory busy, but no more than find a place at once (three to an SM)
+    int chunks = (3 * 148) / max_tiles;
+    chunks = chunks < 1 ? 1 : chunks;
     int per_block = (N + chunks - 1) / chunks;
     per_block = per_block < 8 ? 8 : per_block;
     const dim3 grid(max_tiles, (N + per_block - 1) / per_block), block(256);

@@ -8,8 +8,8 @@
 //     every q and k head turn by the angle position * freq[i] (the angle is an fp32
 //     product, its sine and cosine are taken in fp32); features from R on pass.
 //     q stays in the row; k goes to the token's place in the key pages; every v
-//     head is divided by its root mean square over E (eps under the root) and goes
-//     to the value pages.  Keys and values have sizes of their own (D and E):
+//     head is divided by its root mean square over E (eps under the root; not with a
+//     negative eps) and goes to the value pages.  Keys and values have sizes of their own (D and E):
 //     pages are [page][kv head][token][feature] for each.
 //
 // (2) Attention, one warp per (row, query head), keys one by one in ascending
@@ -74,6 +74,11 @@ __global__ void rotate_norm_append_kernel(T* __restrict__ proj, int proj_stride,
     const T* v_src = row + (size_t)(n_heads + n_kv_heads) * key_dim;
     for (int h = warp; h < n_kv_heads; h += n_warps) {
         const T* v = v_src + (size_t)h * value_dim;
+        if (value_eps < 0.f) {
+            T* as_is = v_cache + v_base + (size_t)h * v_head_stride;
+            for (int e = lane; e < value_dim; e += 32) as_is[e] = v[e];
+            continue;
+        }
         float ss = 0.f;
         for (int e = lane; e < value_dim; e += 32) {
             const float x = cb_to_float(v[e]);

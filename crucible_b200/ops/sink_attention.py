@@ -11,9 +11,10 @@ from . import KernelError, _c_float, _c_int, _check, _code, _need_cuda, _ptr, _s
 
 def rotate_norm_append(proj: torch.Tensor, freq: Optional[torch.Tensor], rotary_dim: int,
                        n_heads: int, n_kv_heads: int, key_dim: int, value_dim: int,
-                       value_eps: float, ctx, cache, binding) -> None:
+                       value_eps: Optional[float], ctx, cache, binding) -> None:
     """Rows of `proj` are [q | k | v | ...]: q and k turn by position * freq (interleaved
-    pairs), q in place; k and the unit-rms v go to the token's place in the pages."""
+    pairs), q in place; k and the unit-rms v (`value_eps` None: v as it is) go to the token's place
+    in the pages."""
     _need_cuda(proj, freq)
     if proj.stride(1) != 1:
         raise KernelError("rotate_norm_append: rows must be contiguous")
@@ -31,7 +32,8 @@ def rotate_norm_append(proj: torch.Tensor, freq: Optional[torch.Tensor], rotary_
         _ptr(ctx.positions), _ptr(ctx.row_request), _ptr(table), _c_int(table.shape[1]),
         _ptr(k_cache), _ptr(v_cache), _c_int(proj.shape[0]), _c_int(n_heads), _c_int(n_kv_heads),
         _c_int(key_dim), _c_int(value_dim), _c_int(cache.page_tokens),
-        _c_int(1 if binding.write else 0), _c_float(value_eps), _stream()), "rotate_norm_append")
+        _c_int(1 if binding.write else 0), _c_float(-1.0 if value_eps is None else value_eps), _stream()),
+        "rotate_norm_append")
 
 
 def norm_rotate_append(proj: torch.Tensor, q_gain: Optional[torch.Tensor], k_gain: Optional[torch.Tensor],

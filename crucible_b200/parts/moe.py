@@ -91,9 +91,12 @@ class MixtureOfExperts(FeedForward):
     # Nothing of a step's routing comes to the host: the launches depend on the step's shape
     # alone, so prompt steps are captured as graphs like decode steps.
     SMALL_MAX_PAIRS = 256        # up to this many pairs the experts' weight rows are read by a warp each
-    SORTED_MIN_PAIRS = 256       # from this many (token, expert) pairs on, a prompt step's experts
-                                 # run as two grouped products over their rows side by side
+    SORTED_MIN_PAIRS = 16        # from this many (token, expert) pairs on, the experts run as two
+                                 # grouped products over their rows side by side (8 experts of 2816 x
+                                 # 2048, two a token: 8 rows 133 us against 152 with a warp per weight
+                                 # row, 16 rows 121 against 259, 64 rows 129 against 784)
     MAX_EXPERTS = 256
+    RIDE_MAX_ROWS = 2            # up to this many bfloat16 rows a gated shared expert rides with the routed ones
 
     def __init__(self, spec: FeedForwardSpec):
         self.spec = spec
@@ -186,12 +189,12 @@ class MixtureOfExperts(FeedForward):
         t, d, f = h.shape[0], self.spec.width, self.ff
         logits = ctx.scratch("moe.logits", (t, self.router.shape[0]), torch.float32)
         ops.linear(h, self.router, logits)
-        # many rows of a prompt: the experts' rows side by side and two grouped products on the
-        # tensor cores, by the plan on the device (tiles of 128 rows); a gated shared expert then
+        # more than a few rows: the experts' rows side by side and two grouped products on the tensor
+        # cores, by the plan on the device (tiles of 128 rows); a gated shared expert then
         # runs as dense products of its own
-        grouped = (self.dtype == torch.bfloat16 and t * self.top >= self.SORTED_MIN_PAIRS
-                   and ctx.host.max_new_tokens > 1 and d % 8 == 0 and f % 8 == 0)
-        riding = 0 if grouped else self.slices
+        grouped = (self.dtype == torch.bfloat16 and d % 8 == 0 and f % 8 == 0
+                   and t * self.top >= self.SORTED_MIN_PAIRS)
+        riding = 0 if grouped or (self.dtype == torch.bfloat16 and t > self.RIDE_MAX_ROWS) else self.slices
         apart = self.shared_gate and not riding
         n, top = self.n + riding, self.top + riding              # experts of the plan, pairs of a token
         tile_rows = kernels.GROUPED_TILE_ROWS if grouped else 0

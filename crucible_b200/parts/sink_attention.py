@@ -111,9 +111,9 @@ class SinkWindowAttention(BranchMixer):
         cache = ctx.cache(binding.group)
         freq, rotary_dim = (self.position.frequencies() if self.position is not None else (None, 0))
         split = bool(getattr(self.position, "split_halves", False))
-        if self.qk_eps is None and not split and self.value_eps is not None:
+        if self.qk_eps is None and not split:
             kernels.rotate_norm_append(proj, freq, rotary_dim, s.n_heads, s.n_kv_heads, s.head_dim,
-                                       self.value_dim, float(self.value_eps), ctx, cache, binding)
+                                       self.value_dim, self.value_eps, ctx, cache, binding)
         else:
             kernels.norm_rotate_append(proj, self.q_gain, self.k_gain,
                                        float(self.qk_eps) if self.qk_eps is not None else 0.0, freq,
