@@ -20,7 +20,13 @@
 
 namespace {
 
-template <typename T>
+// PER neighbouring features, one map's and one head's
+template <typename T, int PER> struct Run { T v[PER]; };
+template <> struct __align__(4) Run<__nv_bfloat16, 2> { __nv_bfloat16 v[2]; };
+template <> struct __align__(8) Run<float, 2> { float v[2]; };
+
+// PER 2: even sizes, rows and pages on boundaries of two elements
+template <typename T, int PER>
 __global__ void differential_prepare_kernel(const T* __restrict__ proj, int proj_stride,
                                             const float* __restrict__ bias, float coef, int every,
                                             const int* __restrict__ positions,
@@ -38,32 +44,36 @@ __global__ void differential_prepare_kernel(const T* __restrict__ proj, int proj
     const int two = 2 * dim, nq = n_heads * two, nk = n_kv_heads * two;
     T* q = qx + (size_t)t * qx_stride;
     // place i of the spread row: query head i / two (head h, map m at 2h + m), feature i % two
-    for (int i = threadIdx.x; i < 2 * nq; i += blockDim.x) {
+    auto take = [&](int src, float factor) {
+        Run<T, PER> r = *reinterpret_cast<const Run<T, PER>*>(row + src);
+#pragma unroll
+        for (int e = 0; e < PER; ++e) {
+            float v = cb_to_float(r.v[e]);
+            if (bias != nullptr) v += bias[src + e];
+            r.v[e] = cb_from_float<T>(v * factor);
+        }
+        return r;
+    };
+    for (int i = threadIdx.x * PER; i < 2 * nq; i += blockDim.x * PER) {
         const int head = i / two, f = i - head * two;
         const int map = head & 1;
-        float v = 0.f;
-        if ((f >= dim) == (map != 0)) {
-            const int src = (head >> 1) * two + f;       // [map 1 | map 2] of head h
-            v = cb_to_float(row[src]);
-            if (bias != nullptr) v += bias[src];
-            v *= temp;
-        }
-        q[i] = cb_from_float<T>(v);
+        Run<T, PER> r;
+#pragma unroll
+        for (int e = 0; e < PER; ++e) r.v[e] = cb_from_float<T>(0.f);
+        if ((f >= dim) == (map != 0)) r = take((head >> 1) * two + f, temp);      // [map 1 | map 2] of head h
+        *reinterpret_cast<Run<T, PER>*>(q + i) = r;
     }
     if (!write_cache) return;
     const int page = block_table[(size_t)row_request[t] * table_stride + pos / page_tokens];
     const size_t at = (size_t)page * n_kv_heads * page_tokens + pos % page_tokens;
-    for (int i = threadIdx.x; i < nk; i += blockDim.x) {
+    for (int i = threadIdx.x * PER; i < nk; i += blockDim.x * PER) {
         const int g = i / two, f = i - g * two;
-        float v = cb_to_float(row[nq + i]);
-        if (bias != nullptr) v += bias[nq + i];
-        k_cache[(at + (size_t)g * page_tokens) * two + f] = cb_from_float<T>(v);
+        *reinterpret_cast<Run<T, PER>*>(k_cache + (at + (size_t)g * page_tokens) * two + f) = take(nq + i, 1.0f);
     }
-    for (int i = threadIdx.x; i < n_kv_heads * value_dim; i += blockDim.x) {
+    for (int i = threadIdx.x * PER; i < n_kv_heads * value_dim; i += blockDim.x * PER) {
         const int g = i / value_dim, f = i - g * value_dim;
-        float v = cb_to_float(row[nq + nk + i]);
-        if (bias != nullptr) v += bias[nq + nk + i];
-        v_cache[(at + (size_t)g * page_tokens) * value_dim + f] = cb_from_float<T>(v);
+        *reinterpret_cast<Run<T, PER>*>(v_cache + (at + (size_t)g * page_tokens) * value_dim + f) =
+            take(nq + nk + i, 1.0f);
     }
 }
 
@@ -107,15 +117,16 @@ CB_EXPORT int cb_differential_prepare(const void* proj, int proj_stride, int dty
     const int places = 4 * n_heads * dim;
     const dim3 block(places >= 2048 ? 512 : (places >= 512 ? 256 : 128));
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == CB_F32)
-        cb_launch(differential_prepare_kernel<float>, dim3(n_rows), block, 0, s, (const float*)proj, proj_stride,
-                  bias, coef, every, positions, row_request, block_table, table_stride, (float*)qx, qx_stride,
-                  (float*)k_cache, (float*)v_cache, n_heads, n_kv_heads, dim, value_dim, page_tokens, write_cache);
-    else
-        cb_launch(differential_prepare_kernel<__nv_bfloat16>, dim3(n_rows), block, 0, s,
-                  (const __nv_bfloat16*)proj, proj_stride, bias, coef, every, positions, row_request, block_table,
-                  table_stride, (__nv_bfloat16*)qx, qx_stride, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache,
-                  n_heads, n_kv_heads, dim, value_dim, page_tokens, write_cache);
+    const uintptr_t unit = dtype == CB_F32 ? 8 : 4;
+    const bool pairs = !((dim | value_dim | proj_stride | qx_stride) & 1) &&
+                       (((uintptr_t)proj | (uintptr_t)qx | (uintptr_t)k_cache | (uintptr_t)v_cache) & (unit - 1)) == 0;
+#define CB_DP(TT, PP)                                                                                          \
+    cb_launch(differential_prepare_kernel<TT, PP>, dim3(n_rows), block, 0, s, (const TT*)proj, proj_stride,    \
+              bias, coef, every, positions, row_request, block_table, table_stride, (TT*)qx, qx_stride,        \
+              (TT*)k_cache, (TT*)v_cache, n_heads, n_kv_heads, dim, value_dim, page_tokens, write_cache)
+    if (dtype == CB_F32) { if (pairs) CB_DP(float, 2); else CB_DP(float, 1); }
+    else { if (pairs) CB_DP(__nv_bfloat16, 2); else CB_DP(__nv_bfloat16, 1); }
+#undef CB_DP
     return cb_last_error();
 }
 

@@ -437,6 +437,12 @@ __global__ void moe_gather_kernel(const T* __restrict__ h, int h_stride, const i
     cb_pdl_wait();
     const T* src = h + (size_t)(sorted_pair[blockIdx.x] / top) * h_stride;
     T* dst = out + (size_t)blockIdx.x * width;
+    constexpr int PER = 16 / sizeof(T);
+    if (width % PER == 0 && h_stride % PER == 0 && (((uintptr_t)h | (uintptr_t)out) & 15) == 0) {
+        for (int i = threadIdx.x * PER; i < width; i += blockDim.x * PER)
+            *reinterpret_cast<uint4*>(dst + i) = *reinterpret_cast<const uint4*>(src + i);
+        return;
+    }
     for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = src[i];
 }
 
@@ -461,7 +467,7 @@ CB_EXPORT int cb_moe_route(const float* logits, int stride, const float* bias, i
         return CB_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     if (E + n_shared > MAX_TOTAL) return CB_ERR_UNSUPPORTED;
-    const int per_warp = n_tokens >= 1024 ? ROUTE_TOKENS : 1, per_block = ROUTE_WARPS * per_warp;
+    const int per_warp = n_tokens >= 16384 ? ROUTE_TOKENS : 1, per_block = ROUTE_WARPS * per_warp;
     cb_launch(moe_route_kernel, dim3((n_tokens + per_block - 1) / per_block), dim3(32 * ROUTE_WARPS), 0, s, logits,
               bias, n_tokens, stride, E, top, idx, weight, place, count, groups, keep, n_shared, gate_col, scale,
               gate_out, per_warp);

@@ -160,7 +160,8 @@ __device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, in
     const int taps = TAPS > 0 ? TAPS : taps_, keep = taps - 1;
     const int lane = threadIdx.x & 31;
     constexpr int W = TAPS > 0 ? TAPS : 1;
-    float past[NV][W], wt[NV][W];
+    // the last inputs of the lane's channels in registers; a token's input is asked for one token ahead
+    float past[NV][W], wt[NV][W], next[NV];
     // the input of channel c0 + lane + 32 i at the portion's token `row` (negative: from the state)
     auto input = [&](int row, int c) {
         return row >= 0 ? cb_to_float(proj[(size_t)(row0 + row) * proj_stride + c])
@@ -176,8 +177,12 @@ __device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, in
                 wt[i][j] = in ? conv_w[(size_t)j * C + c] : 0.f;
                 past[i][j] = (in && j < W - 1) ? input(a - (W - 1) + j, c) : 0.f;
             }
+            next[i] = in ? input(a, c) : 0.f;
         }
     }
+    // (not unrolled: the code of a few tokens' exponentials and divisions does not fit the
+    // instruction cache beside the other units')
+#pragma unroll 1
     for (int t = a; t < b; ++t) {
         float v[NV];
         float ss = 0.f;
@@ -187,7 +192,8 @@ __device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, in
             const bool in = lane + 32 * i < count;
             float acc = 0.f;
             if (TAPS > 0) {
-                past[i][W - 1] = in ? input(t, c) : 0.f;
+                past[i][W - 1] = next[i];
+                next[i] = (in && t + 1 < b) ? input(t + 1, c) : 0.f;
 #pragma unroll
                 for (int j = 0; j < W; ++j) acc = fmaf(wt[i][j], past[i][j], acc);
 #pragma unroll
@@ -195,7 +201,7 @@ __device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, in
             } else if (in) {
                 for (int j = 0; j < taps; ++j) acc = fmaf(conv_w[(size_t)j * C + c], input(t - keep + j, c), acc);
             }
-            v[i] = in ? silu_f(acc) : 0.f;
+            v[i] = __fdividef(acc, 1.0f + expf(-acc));
             ss = fmaf(v[i], v[i], ss);
         }
         float inv = 1.0f;
@@ -216,7 +222,8 @@ __device__ __forceinline__ void channel_conv_unit(const T* __restrict__ proj, in
     }
 }
 
-template <typename T, int TAPS>
+// NQ: pieces of 32 channels of a q or k head (4 for heads up to 128 features, else 8)
+template <typename T, int TAPS, int NQ>
 __global__ void __launch_bounds__(128) channel_delta_prepare_kernel(
     const T* __restrict__ proj, int proj_stride, const float* __restrict__ conv_w, int taps,
     const float* __restrict__ rate, int rate_stride, const float* __restrict__ beta_logit, int beta_stride,
@@ -237,12 +244,8 @@ __global__ void __launch_bounds__(128) channel_delta_prepare_kernel(
     const bool first = blockIdx.y == 0;
     if (unit < 2 * G) {
         const float sc = unit < G ? 1.0f / sqrtf((float)D) : 1.0f;
-        if (D <= 128)
-            channel_conv_unit<T, 4, TAPS>(proj, proj_stride, conv_w, taps, C, unit * D, D, true, sc, tail, row0, n,
-                                          a, b, first, qkv, width);
-        else
-            channel_conv_unit<T, 8, TAPS>(proj, proj_stride, conv_w, taps, C, unit * D, D, true, sc, tail, row0, n,
-                                          a, b, first, qkv, width);
+        channel_conv_unit<T, NQ, TAPS>(proj, proj_stride, conv_w, taps, C, unit * D, D, true, sc, tail, row0, n,
+                                       a, b, first, qkv, width);
         return;
     }
     unit -= 2 * G;
@@ -257,11 +260,30 @@ __global__ void __launch_bounds__(128) channel_delta_prepare_kernel(
     const int d_runs = (H * D + CHANNEL_RUN - 1) / CHANNEL_RUN;
     if (unit < d_runs) {
         const int at = unit * CHANNEL_RUN;
-        for (int i = lane; i < min(CHANNEL_RUN, H * D - at); i += 32) {
-            const float speed = -expf(a_log[(at + i) / D]), bias = dt_bias[at + i];
-            for (int t = a; t < b; ++t)
-                qkv[(size_t)(row0 + t) * width + C + at + i] =
-                    expf(speed * softplus_f(rate[(size_t)(row0 + t) * rate_stride + at + i] + bias));
+        constexpr int N = CHANNEL_RUN / 32;
+        float speed[N], bias[N], next[N];
+        bool in[N];
+        auto logit = [&](int t, int i) { return rate[(size_t)(row0 + t) * rate_stride + at + lane + 32 * i]; };
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int c = at + lane + 32 * i;
+            in[i] = c < H * D;
+            speed[i] = in[i] ? -expf(a_log[c / D]) : 0.f;
+            bias[i] = in[i] ? dt_bias[c] : 0.f;
+            next[i] = in[i] ? logit(a, i) : 0.f;
+        }
+#pragma unroll 1
+        for (int t = a; t < b; ++t) {
+            float z[N];
+#pragma unroll
+            for (int i = 0; i < N; ++i) {
+                z[i] = next[i] + bias[i];
+                next[i] = (in[i] && t + 1 < b) ? logit(t + 1, i) : 0.f;
+            }
+#pragma unroll
+            for (int i = 0; i < N; ++i)
+                if (in[i])
+                    qkv[(size_t)(row0 + t) * width + C + at + lane + 32 * i] = expf(speed[i] * softplus_f(z[i]));
         }
         return;
     }
@@ -874,10 +896,14 @@ CB_EXPORT int cb_channel_delta_prepare(const void* proj, int proj_stride, int dt
     const dim3 grid((n_units + 3) / 4, (max_new + tile - 1) / tile, n_requests), block(128);
     if (grid.y > 65535) return CB_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
-#define CB_CDP(TT, KK)                                                                                      \
-    cb_launch(channel_delta_prepare_kernel<TT, KK>, grid, block, 0, s, (const TT*)proj, proj_stride, conv_w, \
-              taps, rate, rate_stride, beta_logit, beta_stride, a_log, dt_bias, req_row_start,              \
+#define CB_CDP_AS(TT, KK, QQ)                                                                               \
+    cb_launch(channel_delta_prepare_kernel<TT, KK, QQ>, grid, block, 0, s, (const TT*)proj, proj_stride,    \
+              conv_w, taps, rate, rate_stride, beta_logit, beta_stride, a_log, dt_bias, req_row_start,      \
               req_state_slot, (unsigned char*)state, slot_stride, tail_off, qkv, beta, H, G, D, E, n_units, tile)
+#define CB_CDP(TT, KK)                                                                                      \
+    do {                                                                                                    \
+        if (D <= 128) CB_CDP_AS(TT, KK, 4); else CB_CDP_AS(TT, KK, 8);                                      \
+    } while (0)
 #define CB_CDP_TAPS(TT)                                                                                     \
     do {                                                                                                    \
         if (taps == 2) CB_CDP(TT, 2);                                                                       \
@@ -888,6 +914,7 @@ CB_EXPORT int cb_channel_delta_prepare(const void* proj, int proj_stride, int dt
     if (dtype == CB_F32) CB_CDP_TAPS(float); else CB_CDP_TAPS(__nv_bfloat16);
 #undef CB_CDP_TAPS
 #undef CB_CDP
+#undef CB_CDP_AS
     return cb_last_error();
 }
 

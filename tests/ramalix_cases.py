@@ -65,11 +65,11 @@ CASES = {
     # sizes that let the bfloat16 products and attentions run on the tensor cores; the repeated
     # run is the last layer alone
     "ra-c": dict(seed=5, page_tokens=16, config=model(400, 128, 1e-5, 0.4, 2.5, 3, [
-        chunked(4, 2, 64, 64, 0.2, 50, 48, 9000.0, moe(8, 2, 64, (4, 2), 128)),
-        attention(4, 2, 32, 64, 0.3, 0.5, (0.4, 16), moe(4, 2, 72, (2, 2), 72)),
+        chunked(4, 2, 64, 64, 0.1, 50, 48, 9000.0, moe(8, 2, 64, (4, 2), 128)),
+        attention(4, 2, 32, 64, 0.12, 0.5, (0.4, 16), moe(4, 2, 72, (2, 2), 72)),
         delta(4, 1, 64, 32, 4, moe(8, 4, 40, (2, 1), 64)),
-        attention(2, 2, 64, 128, 0.2, 0.2, (0.1, 100), moe(4, 3, 64, None, 24)),
-        chunked(8, 2, 128, 128, 0.1, 96, 64, 9000.0, moe(4, 1, 64, None, None))], (4, 5, 2))),
+        attention(2, 2, 64, 128, 0.08, 0.2, (0.1, 100), moe(4, 3, 64, None, 24)),
+        chunked(8, 2, 128, 128, 0.05, 96, 64, 9000.0, moe(4, 1, 64, None, None))], (4, 5, 2))),
     # no repeated run at all; one tap in both convolutions; keys and values of unlike
     # tensor-core sizes; a chunk longer than any request
     "ra-d": dict(seed=6, page_tokens=32, config=model(150, 48, 1e-6, 1.0, 1.0, 1, [
