@@ -92,7 +92,7 @@ class MixtureOfExperts(FeedForward):
     # alone, so prompt steps are captured as graphs like decode steps.
     SMALL_MAX_PAIRS = 256        # up to this many pairs the experts' weight rows are read by a warp each
     SORTED_MIN_PAIRS = 16        # from this many (token, expert) pairs on, the experts run as two
-                                 # grouped products over their rows side by side (8 experts of 2816 x
+                                 # grouped products over their rows side by side (8 experts of 4096 x
                                  # 2048, two a token: 8 rows 133 us against 152 with a warp per weight
                                  # row, 16 rows 121 against 259, 64 rows 129 against 784)
     MAX_EXPERTS = 256
