@@ -42,8 +42,7 @@ class PositionSpec:
     rotary_dim: int        # how many leading features of a head are rotated
     theta: float
     max_positions: int
-    # options of encodings that stretch their frequencies, as (key, value) pairs:
-    # factor, original, fast, slow
+    # options of encodings that stretch their frequencies, as (key, value) pairs
     scaling: Optional[Tuple[Tuple[str, float], ...]] = None
 
 
@@ -132,12 +131,14 @@ class RunEntry:
     reader reads the copy of the same number).  `add`: (name of one of the model's
     `vectors`, row): that row is added to the residual rows before the layer runs.
     `add_embedding`: the embedding's output (the rows as they were before the first layer)
-    is added to them before that."""
+    is added to them before that.  `project`: the name of one of the model's `matrices` W
+    [width, 2 width]: before any addition the rows become W [x; embedding's output]."""
     layer: int
     cache_of: Optional[int] = None
     copy: int = 0
     add: Optional[Tuple[str, int]] = None
     add_embedding: bool = False
+    project: Optional[str] = None
 
 
 @dataclass(frozen=True)
@@ -155,6 +156,9 @@ class ModelConfig:
     # tables of the model itself, each (name, rows) of float32 rows as wide as the model;
     # a run-order entry may add one of their rows to the residual (`RunEntry.add`)
     vectors: Tuple[Tuple[str, int], ...] = ()
+    # names of the model's matrices [width, 2 width] that a run-order entry may put the rows
+    # and the embedding's output through (`RunEntry.project`)
+    matrices: Tuple[str, ...] = ()
     tensor_names: Mapping[str, str] = field(default_factory=dict, compare=False)
     raw: Mapping[str, Any] = field(default_factory=dict, compare=False)
 
@@ -182,6 +186,9 @@ class ModelConfig:
                 if rows is None or not 0 <= entry.add[1] < rows:
                     raise ConfigError(f"run_order[{i}] adds row {entry.add[1]} of {entry.add[0]!r}, "
                                       f"which the model's vectors do not hold")
+            if entry.project is not None and entry.project not in self.matrices:
+                raise ConfigError(f"run_order[{i}] goes through {entry.project!r}, which the model's "
+                                  f"matrices do not hold")
         for i, layer in enumerate(self.layers):
             names = [name for name, _ in layer.norms]
             if len(set(names)) != len(names):

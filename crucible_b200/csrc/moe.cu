@@ -1,14 +1,16 @@
 // Mixture of experts: every token goes through `top` of `E` small gated feed-forwards,
 //   y[t] = sum_j weight[t][j] * Wd[e_j] (silu(Wg[e_j] h[t]) * (Wu[e_j] h[t])),
 // e_j the experts with the largest router logits of the token (the lower index on equal
-// logits) and weight the softmax over those `top` logits alone.
+// logits) and weight the softmax over those `top` logits alone; or, with sigmoid scores, the experts
+// with the largest sigmoid(logit) + correction, weighted by their sigmoid(logit) as it is.
 //
 // Everything is decided on the device, so a step's launches depend on its shape only:
 //   route    one warp per token: the top logits, their softmax, and each (token, choice)
 //            pair's place among its expert's pairs (a counter per expert); the experts may form
 //            equal groups of neighbours of which only the best few take part (a group's score is
-//            its best logit), and slices of a shared expert may ride along as experts that every
-//            token chooses, weighted by the sigmoid of one logit of the token
+//            its best score or the sum of its two best), and slices of a shared expert may ride
+//            along as experts that every token chooses, weighted by the sigmoid of one logit of the
+//            token or by one
 //   plan     one block: where each expert's pairs start in the sorted order, the list of
 //            row tiles (an expert, a start, a count), and the sorted order itself
 //   tiles    gate/up with the gated pair (SiLU, or the capped form), then down times the pair's weight: a block owns a tile of
@@ -40,12 +42,18 @@ constexpr int ROUTE_WARPS = 8;        // of a routing block ...
 constexpr int ROUTE_TOKENS = 4;       // ... each of which takes up to this many tokens
 constexpr int MAX_TOTAL = 32 * MAX_PER_LANE + 32;      // routed experts and a shared expert's slices
 
+// How a token scores its experts.  sigmoid 0: by their logits, weighted by the softmax over the chosen
+// ones; 1: by sigmoid(logit) + correction (null: nothing), weighted by sigmoid(logit).  best_two: a
+// group's score is the sum of its two best scores instead of its best one.
+struct ScoreRule { int sigmoid, best_two; const float* correction; };
+
 // A pair's place among its expert's pairs: a counter per expert in shared memory, then one addition
 // per block and expert to the global counter.
 __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(
     const float* __restrict__ logits, const float* __restrict__ bias, int n_tokens, int stride, int E, int top,
     int* __restrict__ idx, float* __restrict__ weight, int* __restrict__ place, int* __restrict__ count,
-    int groups, int keep, int n_shared, int gate_col, float scale, float* __restrict__ gate_out, int per_warp) {
+    int groups, int keep, int n_shared, int gate_col, float scale, float* __restrict__ gate_out, int per_warp,
+    ScoreRule rule) {
     cb_pdl_trigger();
     cb_pdl_wait();
     __shared__ float all[ROUTE_WARPS][32 * MAX_PER_LANE], best_of[ROUTE_WARPS][32 * MAX_PER_LANE];
@@ -65,10 +73,12 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(
         for (int i = 0; i < MAX_PER_LANE; ++i) {
             const int e = lane + 32 * i;
             v[i] = e < E ? logits[(size_t)t * stride + e] + (bias != nullptr ? bias[e] : 0.f) : -INFINITY;
+            if (rule.sigmoid && e < E)
+                v[i] = 1.0f / (1.0f + expf(-v[i])) + (rule.correction != nullptr ? rule.correction[e] : 0.f);
         }
         if (keep < groups) {
-            // only the experts of the `keep` groups with the largest best logit (the lower group on
-            // equal ones) stay
+            // only the experts of the `keep` groups with the largest score (the lower group on equal
+            // ones) stay
             const int size = E / groups;
             __syncwarp();
 #pragma unroll
@@ -76,9 +86,13 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(
                 if (lane + 32 * i < E) all[warp][lane + 32 * i] = v[i];
             __syncwarp();
             for (int g = lane; g < groups; g += 32) {
-                float m = -INFINITY;
-                for (int e = g * size; e < (g + 1) * size; ++e) m = fmaxf(m, all[warp][e]);
-                best_of[warp][g] = m;
+                float m = -INFINITY, second = -INFINITY;
+                for (int e = g * size; e < (g + 1) * size; ++e) {
+                    const float s = all[warp][e];
+                    second = fmaxf(second, fminf(m, s));
+                    m = fmaxf(m, s);
+                }
+                best_of[warp][g] = rule.best_two && size > 1 ? m + second : m;
             }
             __syncwarp();
 #pragma unroll
@@ -121,12 +135,14 @@ __global__ void __launch_bounds__(32 * ROUTE_WARPS) moe_route_kernel(
         const size_t at = (size_t)t * (top + n_shared);
         if (lane < top) {
             idx[at + lane] = mine_e;
-            weight[at + lane] = mine / total * scale;
+            weight[at + lane] = (rule.sigmoid
+                ? 1.0f / (1.0f + expf(-(logits[(size_t)t * stride + mine_e] + (bias != nullptr ? bias[mine_e] : 0.f))))
+                : mine / total) * scale;
             chosen[k] = mine_e;
             in_block[k] = atomicAdd(&block_count[mine_e], 1);
         }
-        if (gate_col >= 0) {
-            const float gate = scale / (1.0f + expf(-logits[(size_t)t * stride + gate_col]));
+        if (gate_col >= 0 || n_shared > 0) {
+            const float gate = gate_col >= 0 ? scale / (1.0f + expf(-logits[(size_t)t * stride + gate_col])) : scale;
             // the shared expert's slices: every token's, so its place among their pairs is its own number
             for (int s = lane; s < n_shared; s += 32) {
                 idx[at + top + s] = E + s;
@@ -452,25 +468,26 @@ CB_EXPORT int cb_moe_tile_rows() { return TM; }
 
 // logits: rows at `stride`, the first E of them the experts'.  groups, keep: equal groups of
 // neighbouring experts of which `keep` take part (groups == keep: no restriction).  gate_col >= 0: the
-// column of the shared expert's gate logit; n_shared slices of it ride along as experts E .. E +
-// n_shared - 1 of every token, and gate_out (may be null) receives scale * sigmoid of that logit.
-// scale: on every weight.  count and plan cover E + n_shared experts, a token has top + n_shared pairs.
+// column of the shared expert's gate logit (-1: it has no gate); n_shared slices of it ride along as
+// experts E .. E + n_shared - 1 of every token, and gate_out (may be null) receives scale * sigmoid of
+// that logit.  scale: on every weight.  count and plan cover E + n_shared experts, a token has top +
+// n_shared pairs.  sigmoid, best_two, correction: see ScoreRule.
 CB_EXPORT int cb_moe_route(const float* logits, int stride, const float* bias, int n_tokens, int E, int top,
                            int* idx, float* weight,
                            int* place, int* count, int* plan, int max_tiles, int* sorted_pair,
                            int tile_rows, int groups, int keep, int n_shared, int gate_col, float scale,
-                           float* gate_out, void* stream) {
+                           float* gate_out, int sigmoid, int best_two, const float* correction, void* stream) {
     if (n_tokens <= 0) return 0;
     if (E > 32 * MAX_PER_LANE || top > E || top <= 0 || top > 32) return CB_ERR_UNSUPPORTED;
     if (groups <= 0 || E % groups || keep <= 0 || keep > groups || top > keep * (E / groups) || n_shared < 0 ||
-        (n_shared > 0 && gate_col < 0) || gate_col >= stride)
+        gate_col >= stride)
         return CB_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     if (E + n_shared > MAX_TOTAL) return CB_ERR_UNSUPPORTED;
     const int per_warp = n_tokens >= 16384 ? ROUTE_TOKENS : 1, per_block = ROUTE_WARPS * per_warp;
     cb_launch(moe_route_kernel, dim3((n_tokens + per_block - 1) / per_block), dim3(32 * ROUTE_WARPS), 0, s, logits,
               bias, n_tokens, stride, E, top, idx, weight, place, count, groups, keep, n_shared, gate_col, scale,
-              gate_out, per_warp);
+              gate_out, per_warp, ScoreRule{sigmoid, best_two, correction});
     cb_launch(moe_plan_kernel, dim3(1), dim3(n_tokens * (top + n_shared) > 256 ? 1024 : 256), 0, s, count, E + n_shared, n_tokens * (top + n_shared),
               (const int*)idx, (const int*)place, plan, max_tiles, sorted_pair, tile_rows > 0 ? tile_rows : TM);
     return cb_last_error();

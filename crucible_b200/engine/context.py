@@ -172,6 +172,22 @@ class StepContext:
     _announced = None            # (norm, address and shape of the rows it will read)
     _offer = None                # (norm, address and shape of the rows, scaled, sumsq, parts)
 
+    # -- norms taken where a layer ends ---------------------------------------
+    # An arrangement that ends its layer with one launch over the residual may take the norms
+    # of what reads the rows next in that launch (into scratch rows both sides know) and offer
+    # them; the reader takes the offer instead of a launch of its own.
+    norms_after_layer = None     # set by the model before each layer: the norms that read the
+                                 # rows after it, of a reader that knows such an offer, or None
+    _closed = None               # (norms, address and shape of the rows)
+
+    def offer_closed(self, rows: torch.Tensor, norms) -> None:
+        self._closed = (tuple(norms), rows.data_ptr(), tuple(rows.shape))
+
+    def take_closed(self, rows: torch.Tensor, norms) -> bool:
+        o, self._closed = self._closed, None
+        return (o is not None and len(o[0]) == len(norms) and all(a is b for a, b in zip(o[0], norms))
+                and o[1] == rows.data_ptr() and o[2] == tuple(rows.shape))
+
     def announce_norm(self, norm, rows: Optional[torch.Tensor]) -> None:
         self._announced = (norm, rows.data_ptr(), tuple(rows.shape)) if norm is not None else None
         self._offer = None

@@ -19,6 +19,7 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from .. import ops
+from ..ops import layer_close
 from ..config.model_config import ConfigError, ModelConfig
 from ..parts import (ARRANGEMENTS, EMBEDDINGS, FEED_FORWARDS, HEADS, MIXERS, NORMS, CacheNeed,
                      LayerBinding, TensorDecl)
@@ -59,6 +60,40 @@ class ModelVectors:
         return self.bound[name][index]
 
 
+class ModelMatrices:
+    """Matrices of the model itself, W [width, 2 width] by name: a run-order entry may put the
+    residual x and the embedding's output x0 through one of them, x <- W [x; x0].  The part of
+    the product that x0 has is the same whenever it is taken, so a step takes it once."""
+
+    def __init__(self, names, width: int):
+        self.names = tuple(names)
+        self.width = width
+        self.halves: Dict[str, Tuple[torch.Tensor, torch.Tensor]] = {}
+
+    def tensors(self):
+        return [TensorDecl(name, (self.width, 2 * self.width)) for name in self.names]
+
+    def bind(self, tensors, dtype, device):
+        self.dtype = dtype
+        for name in self.names:
+            w = tensors[name]
+            self.halves[name] = (w[:, :self.width].contiguous(), w[:, self.width:].contiguous())
+            ops.declare_weights(*self.halves[name])
+
+    def of_embedding(self, ctx, name: str, x: torch.Tensor) -> torch.Tensor:
+        """The embedding's share of every later `enter`; `x`: the embedding's output."""
+        rows = ctx.scratch("entry.rows", x.shape, self.dtype)
+        layer_close.swap_rows(x, rows)
+        share = ctx.scratch(f"entry.share.{name}", x.shape, torch.float32)
+        ops.linear(rows, self.halves[name][1], share)
+        return share
+
+    def enter(self, ctx, name: str, x: torch.Tensor, share: torch.Tensor) -> None:
+        rows = ctx.scratch("entry.rows", x.shape, self.dtype)
+        layer_close.swap_rows(x, rows, share)
+        ops.linear(rows, self.halves[name][0], x, accumulate=True)
+
+
 class DecoderModel:
     def __init__(self, config: ModelConfig):
         self.config = config
@@ -68,6 +103,7 @@ class DecoderModel:
                                 config.hidden_size, config.tie_word_embeddings)
         self.final_norm = NORMS.build(config.final_norm.kind, config.final_norm)
         self.vectors = ModelVectors(config.vectors, config.hidden_size)
+        self.matrices = ModelMatrices(config.matrices, config.hidden_size)
         self.layers = []
         for spec in config.layers:
             mixer = MIXERS.build(spec.mixer.kind, spec.mixer)
@@ -162,6 +198,8 @@ class DecoderModel:
         yield "final_norm", self.final_norm, None
         if self.vectors.tables:
             yield "vectors", self.vectors, None
+        if self.matrices.names:
+            yield "matrices", self.matrices, None
         for li, layer in enumerate(self.layers):
             for name, norm in layer.norms.items():
                 yield f"layer.{name}", norm, li
@@ -233,20 +271,27 @@ class DecoderModel:
         if any(entry.add_embedding for entry in order):
             embedded = ctx.scratch("embedding.output", x.shape, torch.float32)
             embedded.copy_(x)
+        shares = {name: self.matrices.of_embedding(ctx, name, x)
+                  for name in self.matrices.names if any(entry.project == name for entry in order)}
         for i, (entry, binding) in enumerate(zip(order, self.bindings)):
             # the norm that reads the rows after this layer, for the layer's last product
             nxt = self.layers[order[i + 1].layer] if i + 1 < len(order) else None
             entry_norm = getattr(nxt, "entry_norm", None)
             # (rows that get a vector added before the next layer are not final when this one ends)
-            changed = i + 1 < len(order) and (order[i + 1].add is not None or order[i + 1].add_embedding)
+            changed = i + 1 < len(order) and (order[i + 1].add is not None or order[i + 1].add_embedding
+                                              or order[i + 1].project is not None)
             ctx.norm_after_layer = entry_norm() if entry_norm is not None and not changed else None
+            norms_at_entry = getattr(nxt, "norms_at_entry", None)
+            ctx.norms_after_layer = norms_at_entry() if norms_at_entry is not None and not changed else None
+            if entry.project is not None:
+                self.matrices.enter(ctx, entry.project, x, shares[entry.project])
             vector = self.vectors.row(*entry.add) if entry.add is not None else None
             if entry.add_embedding:
                 ops.add_rows(x, embedded, vector)
             elif vector is not None:
                 ops.add_vector(x, vector)
             self.layers[entry.layer].forward(ctx, x, binding)
-        ctx.norm_after_layer = None
+        ctx.norm_after_layer = ctx.norms_after_layer = None
         if ctx.n_logit_rows == 0:
             return ctx.scratch("logits", (0, self.config.vocab_size), torch.float32)
         if x.dim() == 3:

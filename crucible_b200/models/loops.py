@@ -2,7 +2,9 @@
 `loop` = {`start`, `stop`, `times`}: the layers start .. stop - 1 run `times` times in a row with
 the same weights, each pass a copy with keys and state of its own; row t of the model's table
 `LOOP_VECTORS` is added to the residual before pass t.  `embedding_again`: the embedding's output
-is added to it before every pass but the first, ahead of the row."""
+is added to it before every pass but the first, ahead of the row.  `project`: instead of the rows of
+`LOOP_VECTORS`, every pass begins with x <- W [x; embedding's output], W the model's matrix
+`LOOP_MATRIX`."""
 from __future__ import annotations
 
 from typing import Any, Mapping
@@ -10,6 +12,7 @@ from typing import Any, Mapping
 from ..config.model_config import ConfigError, KeyReader, RunEntry
 
 LOOP_VECTORS = "loop_step"      # the model's table of the vectors added before each pass
+LOOP_MATRIX = "loop_in"         # the model's matrix that the rows go through before each pass
 
 
 def _count(raw: Mapping[str, Any], key: str, where: str) -> int:
@@ -19,8 +22,8 @@ def _count(raw: Mapping[str, Any], key: str, where: str) -> int:
     return v
 
 
-def looped_run_order(raw: Mapping[str, Any], n_layers: int, embedding_again: bool = False):
-    """(run order, rows of the passes' vectors: 0 without a `loop`)."""
+def looped_run_order(raw: Mapping[str, Any], n_layers: int, embedding_again: bool = False, project: bool = False):
+    """(run order, number of passes: 0 without a `loop`)."""
     loop = raw.get("loop")
     if loop is None:
         return tuple(RunEntry(layer=i) for i in range(n_layers)), 0
@@ -36,7 +39,8 @@ def looped_run_order(raw: Mapping[str, Any], n_layers: int, embedding_again: boo
         return tuple(RunEntry(layer=i) for i in range(n_layers)), times
     order = [RunEntry(layer=i) for i in range(start)]
     for t in range(times):
-        order += [RunEntry(layer=i, copy=t, add=(LOOP_VECTORS, t) if i == start else None,
+        order += [RunEntry(layer=i, copy=t, add=(LOOP_VECTORS, t) if i == start and not project else None,
+                           project=LOOP_MATRIX if i == start and project else None,
                            add_embedding=embedding_again and i == start and t > 0)
                   for i in range(start, stop)]
     order += [RunEntry(layer=i) for i in range(stop, n_layers)]

@@ -52,6 +52,7 @@ MODULES: Dict[str, List[str]] = {
     "moe": ["common.cuh"],
     "input_conv": ["common.cuh"],
     "differential": ["common.cuh"],
+    "layer_close": ["common.cuh"],
 }
 
 _loaded: Dict[str, ctypes.CDLL] = {}

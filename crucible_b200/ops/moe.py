@@ -34,7 +34,8 @@ def _pair(pair):
 
 def route(logits, top: int, idx, weight, place, count, plan, tiles: int, sorted_pair, bias=None,
           rows: int = 0, n_experts: int = 0, groups=None, n_shared: int = 0, gate_col: int = -1,
-          scale: float = 1.0, gate_out=None) -> None:
+          scale: float = 1.0, gate_out=None, sigmoid: bool = False, correction=None,
+          group_best_two: bool = False) -> None:
     """Per token the `top` largest logits (plus `bias`, float32 [experts], if given; the lower
     index on ties) and their softmax; then
     the sorted order of the (token, choice) pairs by expert and the tiles (of `rows` rows; 0: this
@@ -45,14 +46,20 @@ def route(logits, top: int, idx, weight, place, count, plan, tiles: int, sorted_
     logits take part.  `n_shared` slices of a shared expert ride along as further experts (after the
     routed ones) that every token chooses, weighted by the sigmoid of logit `gate_col`; `gate_out`
     (float32 [tokens] or None) receives that weight.  `scale`: on every weight.  `count` and the plan
-    cover the slices too, and a token has top + n_shared pairs."""
-    _need_cuda(logits, idx, weight, place, count, plan, sorted_pair, bias, gate_out)
+    cover the slices too, and a token has top + n_shared pairs; `gate_col` -1: their weight is `scale`.
+    `sigmoid`: experts are chosen by sigmoid(logit) + `correction` (float32 [experts] or None) and
+    weighted by sigmoid(logit), not by a softmax.  `group_best_two`: a group's score is the sum of its
+    two best instead of its best."""
+    _need_cuda(logits, idx, weight, place, count, plan, sorted_pair, bias, gate_out, correction)
     if logits.dtype != torch.float32 or not logits.is_contiguous():
         raise KernelError("moe route takes contiguous float32 logits [tokens, experts]")
     t, e = logits.shape[0], n_experts or logits.shape[1]
     pairs, total = t * (top + n_shared), e + n_shared
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != e or not bias.is_contiguous()):
         raise KernelError("moe route: the bias is float32 [experts]")
+    if correction is not None and (not sigmoid or correction.dtype != torch.float32 or correction.numel() != e
+                                   or not correction.is_contiguous()):
+        raise KernelError("moe route: the correction is float32 [experts], for sigmoid scores")
     if (idx.numel() < pairs or plan.numel() < plan_ints(total, tiles) or sorted_pair.numel() < pairs
             or count.numel() < total):
         raise KernelError("moe route: a buffer is too small")
@@ -61,7 +68,8 @@ def route(logits, top: int, idx, weight, place, count, plan, tiles: int, sorted_
     _check(lib.cb_moe_route(_ptr(logits), _c_int(logits.shape[1]), _ptr(bias), _c_int(t), _c_int(e), _c_int(top),
                             _ptr(idx), _ptr(weight), _ptr(place), _ptr(count), _ptr(plan), _c_int(tiles),
                             _ptr(sorted_pair), _c_int(rows), _c_int(count_g), _c_int(keep_g), _c_int(n_shared),
-                            _c_int(gate_col), ctypes.c_float(scale), _ptr(gate_out), _stream()), "moe route")
+                            _c_int(gate_col), ctypes.c_float(scale), _ptr(gate_out), _c_int(1 if sigmoid else 0),
+                            _c_int(1 if group_best_two else 0), _ptr(correction), _stream()), "moe route")
 
 
 def expert_tiles(gated: bool, a, w, n_out: int, plan, n_experts: int, tiles: int, sorted_pair, top: int,

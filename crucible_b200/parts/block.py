@@ -1,9 +1,12 @@
 """Block arrangements.  `pre_norm` is the only one the reference runs on the
 GPU (`model.py:262-264`, `engine/src/gpu_model.rs:518-520`):
 x = x + mixer(norm(x)); x = x + ffn(norm(x)).  `parallel` has one norm that both
-sublayers read: with n = norm(x), x = x + mixer(n) + ffn(n).  `pre_norm_conv` is `pre_norm`
+sublayers read: with n = norm(x), x = x + mixer(n) + ffn(n).  `parallel_two_norms` gives each of
+the two a norm of its own over the same x and may scale their results.  `pre_norm_conv` is `pre_norm`
 with a short causal convolution on what each sublayer reads."""
 from __future__ import annotations
+
+import torch
 
 from .base import ARRANGEMENTS, Arrangement, TensorDecl
 
@@ -80,6 +83,70 @@ class ParallelBlock(Arrangement):
             self.feed_forward.forward(ctx, n, x)
 
 
+class ParallelTwoNormBlock(Arrangement):
+    """x += s1 * mixer(mixer_norm(x)) + s2 * ffn(feed_forward_norm(x)), both norms of the same x.
+    Option `layer_scale` of the layer: s1 and s2 are the float32 vectors `mixer_scale` and
+    `feed_forward_scale` [width] (else ones).  The mixer writes its result beside the residual and
+    the feed-forward leaves its sum open; one launch adds both in 32 bits and takes the norms of
+    the layer that follows.  The mixer must be able to write instead of add (`can_overwrite`), the
+    feed-forward must offer `forward_open`, or be absent."""
+    norm_names = ("mixer_norm", "feed_forward_norm")
+
+    def __init__(self, spec, norms, mixer, feed_forward):
+        self.has_ffn = not getattr(feed_forward, "absent", False)
+        if not self.has_ffn:
+            self.norm_names = ("mixer_norm",)
+        super().__init__(spec, norms, mixer, feed_forward)
+        if not getattr(mixer, "can_overwrite", False):
+            raise ValueError("parallel_two_norms: the mixer must be able to write its result")
+        if self.has_ffn and not hasattr(feed_forward, "forward_open"):
+            raise ValueError("parallel_two_norms: the feed-forward must leave its sum open")
+        self.width = spec.mixer.width
+        self.scaled = bool(spec.option("layer_scale", False))
+        self.scales = {}
+
+    def tensors(self):
+        if not self.scaled:
+            return []
+        return [TensorDecl(f"{name}_scale", (self.width,), role="vector", init=("normal", 0.8, 0.2))
+                for name in (("mixer", "feed_forward") if self.has_ffn else ("mixer",))]
+
+    def bind(self, tensors, dtype, device):
+        self.scales = {name: t.contiguous() for name, t in tensors.items() if t is not None}
+
+    def norms_at_entry(self):
+        """The norms that read the rows this layer is given, in the order of `norm_names`."""
+        return tuple(self.norms[name] for name in self.norm_names)
+
+    def forward(self, ctx, x, binding):
+        from ..ops import layer_close
+        announce = getattr(ctx, "announce_norm", None)
+        if announce is not None:
+            announce(None, None)
+        mine = self.norms_at_entry()
+        if ctx.take_closed(x, mine):
+            h = self._rows(ctx, x, mine)
+        else:
+            h = self._rows(ctx, x, mine)
+            layer_close.close(x, None, None, None, None, self._norm_args(mine, h))
+        mixed = ctx.scratch("layer.mixed", x.shape, torch.float32)
+        self.mixer.forward(ctx, h[0], mixed, binding, accumulate=False)
+        left = self.feed_forward.forward_open(ctx, h[1]) if self.has_ffn else None
+        after = getattr(ctx, "norms_after_layer", None) or ()
+        layer_close.close(x, mixed, self.scales.get("mixer_scale"), left, self.scales.get("feed_forward_scale"),
+                          self._norm_args(after, self._rows(ctx, x, after)))
+        if after:
+            ctx.offer_closed(x, after)
+
+    @staticmethod
+    def _rows(ctx, x, norms):
+        return [ctx.scratch(f"layer.normed{i}", x.shape, norm.dtype) for i, norm in enumerate(norms)]
+
+    @staticmethod
+    def _norm_args(norms, rows):
+        return [(norm.gain, norm.spec.eps, out) for norm, out in zip(norms, rows)]
+
+
 class PreNormConvBlock(PreNormBlock):
     """x += mixer(c1(norm(x))); x += ffn(c2(norm(x))), c(h)_t = h_t + sum_j w_j h_(t - taps + 1 + j)
     along a request's tokens, channel by channel (zeros before its start).  Norm, convolution and
@@ -139,3 +206,4 @@ class PreNormConvBlock(PreNormBlock):
 ARRANGEMENTS.register("pre_norm", PreNormBlock)
 ARRANGEMENTS.register("pre_norm_conv", PreNormConvBlock)
 ARRANGEMENTS.register("parallel", ParallelBlock)
+ARRANGEMENTS.register("parallel_two_norms", ParallelTwoNormBlock)

@@ -16,7 +16,11 @@ logits are h Wr^T + b, tensor `router.b`), `pair` = (limit, alpha, offset): the 
 the capped gated pair instead of silu(g) * u; `groups` = (count, keep): the experts form `count`
 equal groups of neighbours, a group's score is its best logit, and only the experts of the `keep`
 best groups can be chosen; `shared_gate` (tensor `shared.sg` [1, width]): the shared expert's result
-is multiplied by sigmoid(h Wsg^T), one number a token; `out_scale`: everything times this number.
+is multiplied by sigmoid(h Wsg^T), one number a token; `out_scale`: everything times this number;
+`score` = "sigmoid": with s = sigmoid(z) the experts with the largest s + `correction` (a float32
+vector) are chosen and weighted by s as it is; `group_score` = "two_best": a group's score is the sum
+of its two best scores (default "best").  `forward_open` leaves the sum to the caller (an arrangement
+that scales it and adds a mixer's result in the same pass), the shared expert included.
 (The softmax over the chosen logits alone is the chosen experts' softmax over all experts divided
 by their sum.)
 """
@@ -27,6 +31,7 @@ import torch
 from .. import ops
 from ..config.model_config import FeedForwardSpec
 from ..ops import moe as kernels
+from ..ops.layer_close import OpenSum
 from .base import FEED_FORWARDS, FeedForward, TensorDecl
 from .swiglu import SwiGLU
 
@@ -96,7 +101,7 @@ class MixtureOfExperts(FeedForward):
                                  # 2048, two a token: 8 rows 133 us against 152 with a warp per weight
                                  # row, 16 rows 121 against 259, 64 rows 129 against 784)
     MAX_EXPERTS = 256
-    RIDE_MAX_ROWS = 2            # up to this many bfloat16 rows a gated shared expert rides with the routed ones
+    RIDE_MAX_ROWS = 2            # up to this many bfloat16 rows a joining shared expert rides with the routed ones
 
     def __init__(self, spec: FeedForwardSpec):
         self.spec = spec
@@ -107,6 +112,11 @@ class MixtureOfExperts(FeedForward):
         self.has_bias = bool(spec.option("router_bias", False))
         self.shared_gate = bool(spec.option("shared_gate", False))
         self.out_scale = float(spec.option("out_scale", 1.0))
+        self.score = str(spec.option("score", "softmax"))
+        self.group_score = str(spec.option("group_score", "best"))
+        if self.score not in ("softmax", "sigmoid") or self.group_score not in ("best", "two_best"):
+            raise ValueError(f"moe: score is 'softmax' or 'sigmoid', group_score 'best' or 'two_best', got "
+                             f"{self.score!r} and {self.group_score!r}")
         groups = spec.option("groups")
         self.groups = (int(groups[0]), int(groups[1])) if groups is not None else None
         pair = spec.option("pair")
@@ -127,12 +137,17 @@ class MixtureOfExperts(FeedForward):
         if shared and not self.shared_gate and self.out_scale != 1.0:
             raise ValueError("moe: a shared expert without a gate takes no out_scale")
         self.shared_ff = int(shared) if shared else 0
-        self.shared = (SwiGLU(FeedForwardSpec(kind="swiglu", width=spec.width, intermediate=self.shared_ff))
-                       if shared and not self.shared_gate else None)
         self.shared_gate = self.shared_gate and self.shared_ff > 0
-        # A gated shared expert as slices of an expert's size (the last one padded with zeros) that
+        # a shared expert that joins the experts' sum: one with a gate, or one of a caller that
+        # takes the sum open
+        self.joins = self.shared_ff > 0 and (self.shared_gate or bool(spec.option("open_sum", False)))
+        if self.joins and self.pair is not None:
+            raise ValueError("moe: a shared expert that joins the experts' sum has no capped pair")
+        self.shared = (SwiGLU(FeedForwardSpec(kind="swiglu", width=spec.width, intermediate=self.shared_ff))
+                       if shared and not self.joins else None)
+        # A joining shared expert as slices of an expert's size (the last one padded with zeros) that
         # every token chooses: a few rows then take no launches of their own for it.
-        self.slices = -(-self.shared_ff // self.ff) if self.shared_gate else 0
+        self.slices = -(-self.shared_ff // self.ff) if self.joins else 0
         if self.slices > 32 or self.n + self.slices > self.MAX_EXPERTS:
             self.slices = 0
 
@@ -141,15 +156,19 @@ class MixtureOfExperts(FeedForward):
         out = [TensorDecl("router", (self.n, d))]
         if self.has_bias:
             out.append(TensorDecl("router.b", (self.n,), role="vector", init=("normal", 0.0, 0.5)))
+        if self.score == "sigmoid":
+            out.append(TensorDecl("correction", (self.n,), role="vector", init=("normal", 0.0, 0.5)))
         for e in range(self.n):
             out += [TensorDecl(f"e{e}.gate", (f, d)), TensorDecl(f"e{e}.up", (f, d)),
                     TensorDecl(f"e{e}.down", (d, f))]
         if self.shared is not None:
             out += [TensorDecl(f"shared.{t.name}", t.shape, t.role) for t in self.shared.tensors()]
-        elif self.shared_gate:
+        elif self.joins:
             fs = self.shared_ff
             out += [TensorDecl("shared.gate", (fs, d)), TensorDecl("shared.up", (fs, d)),
-                    TensorDecl("shared.down", (d, fs)), TensorDecl("shared.sg", (1, d))]
+                    TensorDecl("shared.down", (d, fs))]
+            if self.shared_gate:
+                out.append(TensorDecl("shared.sg", (1, d)))
         return out
 
     def bind(self, tensors, dtype, device):
@@ -159,6 +178,7 @@ class MixtureOfExperts(FeedForward):
         self.router = (torch.cat([tensors["router"], tensors["shared.sg"]], 0).contiguous()
                        if self.shared_gate else tensors["router"])
         self.router_bias = tensors.get("router.b") if self.has_bias else None
+        self.correction = tensors.get("correction") if self.score == "sigmoid" else None
         gate_up = [torch.cat([tensors[f"e{e}.gate"], tensors[f"e{e}.up"]], 0) for e in range(self.n)]
         down = [tensors[f"e{e}.down"] for e in range(self.n)]
         for s in range(self.slices):
@@ -173,7 +193,7 @@ class MixtureOfExperts(FeedForward):
         ops.declare_weights(self.router, self.gate_up, self.down)
         # the shared expert as dense products, for steps of many rows
         self.dense = []
-        if self.shared_gate:
+        if self.joins:
             if self.slices:
                 self.dense = [(self.gate_up[self.n + s], self.down[self.n + s]) for s in range(self.slices)]
             else:
@@ -186,16 +206,23 @@ class MixtureOfExperts(FeedForward):
                              dtype, device)
 
     def forward(self, ctx, h, residual):
+        o = self.forward_open(ctx, h)
+        kernels.combine(o.rows, o.top, residual, by_plan=o.by_plan, shared=o.shared, gate=o.gate)
+        if self.shared is not None:
+            self.shared.forward(ctx, h, residual)
+
+    def forward_open(self, ctx, h) -> OpenSum:
+        """The experts' rows and what the shared expert adds if it joins their sum, not yet summed."""
         t, d, f = h.shape[0], self.spec.width, self.ff
         logits = ctx.scratch("moe.logits", (t, self.router.shape[0]), torch.float32)
         ops.linear(h, self.router, logits)
         # more than a few rows: the experts' rows side by side and two grouped products on the tensor
-        # cores, by the plan on the device (tiles of 128 rows); a gated shared expert then
+        # cores, by the plan on the device (tiles of 128 rows); a joining shared expert then
         # runs as dense products of its own
         grouped = (self.dtype == torch.bfloat16 and d % 8 == 0 and f % 8 == 0
                    and t * self.top >= self.SORTED_MIN_PAIRS)
         riding = 0 if grouped or (self.dtype == torch.bfloat16 and t > self.RIDE_MAX_ROWS) else self.slices
-        apart = self.shared_gate and not riding
+        apart = self.joins and not riding
         n, top = self.n + riding, self.top + riding              # experts of the plan, pairs of a token
         tile_rows = kernels.GROUPED_TILE_ROWS if grouped else 0
         tiles = kernels.max_tiles(t, top, n, tile_rows)
@@ -204,10 +231,12 @@ class MixtureOfExperts(FeedForward):
         order = ctx.scratch("moe.order", (t * top,), torch.int32)
         weight = ctx.scratch("moe.weight", (t * top,), torch.float32)
         plan = ctx.scratch("moe.plan", (kernels.plan_ints(n, tiles),), torch.int32)
-        gate = ctx.scratch("moe.shared_gate", (t,), torch.float32) if apart else None
+        gate = ctx.scratch("moe.shared_gate", (t,), torch.float32) if apart and self.shared_gate else None
         kernels.route(logits, self.top, idx, weight, place, self.count, plan, tiles, order, bias=self.router_bias,
                       rows=tile_rows, n_experts=self.n, groups=self.groups, n_shared=riding,
-                      gate_col=self.n if self.shared_gate else -1, scale=self.out_scale, gate_out=gate)
+                      gate_col=self.n if self.shared_gate else -1, scale=self.out_scale, gate_out=gate,
+                      sigmoid=self.score == "sigmoid", correction=self.correction,
+                      group_best_two=self.group_score == "two_best")
         act = ctx.scratch("moe.act", (t * top, f), self.dtype)
         by_plan = None
         if grouped:
@@ -236,9 +265,7 @@ class MixtureOfExperts(FeedForward):
                 shared_act = ctx.scratch("moe.shared_act", (t, down.shape[1]), self.dtype)
                 ops.linear_swiglu(h, gate_up, shared_act, ctx)
                 ops.linear(shared_act, down, shared_out, accumulate=i > 0)
-        kernels.combine(pair_out, top, residual, by_plan=by_plan, shared=shared_out, gate=gate)
-        if self.shared is not None:
-            self.shared.forward(ctx, h, residual)
+        return OpenSum(rows=pair_out, top=top, by_plan=by_plan, shared=shared_out, gate=gate)
 
 
 FEED_FORWARDS.register("dense_act", ActivatedFeedForward)

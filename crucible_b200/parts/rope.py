@@ -8,6 +8,8 @@ The tables are fp32 in both engine dtypes and the rotation is fp32 arithmetic.
 """
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..config.model_config import PositionSpec
@@ -57,7 +59,12 @@ class InterleavedRotary(PositionEncoding):
     turn by the angle position * theta^(-2i / rotary_dim); features from rotary_dim on
     pass unchanged.  (u, v) -> (u cos a - v sin a, v cos a + u sin a).  The frequencies
     are float32 numbers and the angle is a float32 product taken in the kernel, so there
-    is no table over positions and no longest position."""
+    is no table over positions and no longest position.
+
+    With the options `factor`, `low`, `high`, `original` (the spec's `scaling`) the frequencies are
+    stretched by wavelength l = 2 pi / f, as in Llama 3.1: f stays where l < original / high, becomes
+    f / factor where l > original / low, and between the two is (1 - s) f / factor + s f with
+    s = (original / l - low) / (high - low)."""
 
     split_halves = False       # which features pair: neighbours (2i, 2i + 1)
 
@@ -65,13 +72,28 @@ class InterleavedRotary(PositionEncoding):
         if spec.rotary_dim % 2 != 0 or spec.rotary_dim < 0:
             raise ValueError(f"rotary_dim must be even and not negative, got {spec.rotary_dim}")
         self.spec = spec
+        self.scaling = dict(spec.scaling) if spec.scaling else None
+        if self.scaling is not None and set(self.scaling) != {"factor", "low", "high", "original"}:
+            raise ValueError("rope_interleaved: the stretched frequencies need 'factor', 'low', 'high' and 'original'")
         self.freq = None
 
-    def bind(self, tensors, dtype, device):
+    def _frequencies(self) -> torch.Tensor:
         n = self.spec.rotary_dim
         i = torch.arange(n // 2, dtype=torch.float64)
+        f = float(self.spec.theta) ** (-2.0 * i / n)
+        if self.scaling is not None:
+            sc = self.scaling
+            length = 2.0 * math.pi / f
+            slow = f / sc["factor"]
+            s = (sc["original"] / length - sc["low"]) / (sc["high"] - sc["low"]) if sc["high"] != sc["low"] else 1.0
+            between = (1.0 - s) * slow + s * f
+            f = torch.where(length < sc["original"] / sc["high"], f,
+                            torch.where(length > sc["original"] / sc["low"], slow, between))
+        return f
+
+    def bind(self, tensors, dtype, device):
         # taken in float64 and rounded once, so every frequency is the nearest float32
-        self.freq = (float(self.spec.theta) ** (-2.0 * i / n)).to(torch.float32).to(device) if n else None
+        self.freq = self._frequencies().to(torch.float32).to(device) if self.spec.rotary_dim else None
 
     def frequencies(self):
         return self.freq, self.spec.rotary_dim

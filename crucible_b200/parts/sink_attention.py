@@ -11,7 +11,8 @@ exp(s_j - m) + exp(sink_i - m)): the sink of head i has no key and no value and 
 scaled.  The heads' results times sigmoid(h Wg^T) go through Wo.
 
 Options of the spec: value_dim (default head_dim), keep_first (default 0), sink
-(default true), value_norm_eps (None: values are cached as they are), gate (default
+(default true: learned, `sink` [H]; a number: every head's sink has that score, 0 adds one to the
+denominator; false: none), value_norm_eps (None: values are cached as they are), gate (default
 true or "element": a logit for every output feature, `g` [H * E, width]; "head": one logit a
 head, `g` [H, width]; false: none), qk_norm_eps (default None; a number: every q and k head is
 divided by its root mean square over D, that eps under the root, and multiplied by the weight
@@ -50,7 +51,9 @@ class SinkWindowAttention(BranchMixer):
         self.spec = spec
         self.value_dim = int(spec.option("value_dim", spec.head_dim))
         self.keep_first = int(spec.option("keep_first", 0))
-        self.has_sink = bool(spec.option("sink", True))
+        sink = spec.option("sink", True)
+        self.fixed_sink = float(sink) if sink is not None and not isinstance(sink, bool) else None
+        self.has_sink = sink is True
         gate = spec.option("gate", True)
         self.gate = {True: "element", False: None, None: None}.get(gate, gate)
         if self.gate not in (None, "element", "head"):
@@ -93,6 +96,8 @@ class SinkWindowAttention(BranchMixer):
         self.w_in = torch.cat(parts, dim=0).contiguous()
         self.w_out = tensors["o"]
         self.sinks = tensors.get("sink") if self.has_sink else None
+        if self.fixed_sink is not None:
+            self.sinks = torch.full((self.spec.n_heads,), self.fixed_sink, dtype=torch.float32, device=device)
         self.q_gain = tensors.get("q.norm") if self.qk_eps is not None else None
         self.k_gain = tensors.get("k.norm") if self.qk_eps is not None else None
         self.dtype = dtype
