@@ -188,3 +188,28 @@ def ramalix(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, vocab
 
 SHAPES["ramalix-w1024"] = ramalix(*COMPARISON_SIZES["w1024"])
 SHAPES["ramalix-w2048"] = ramalix(*COMPARISON_SIZES["w2048"])
+
+
+def gavipel(width: int, heads: int, kv_heads: int, head_dim: int, ff: int, vocab: int,
+            layers: int = 4, experts: int = 8, top: int = 2, window: int = 1024, passes: int = 1) -> dict:
+    """A Gavipel config.json of a real model's proportions: every layer is windowed attention
+    (`heads * head_dim` wide, half of each head turned, the rotation stretched beyond 8,192 positions)
+    beside `experts` experts of half the dense width in four groups of which two take part, a token
+    using `top` of them and a shared expert of the same size.  Layers 1 and 2 form the repeated run,
+    `passes` times (1: every layer runs once)."""
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": ff // 2}, "shared": {"ff": ff // 2}}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                 "rot": {"base": 500000.0, "dims": head_dim // 2,
+                         "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}},
+                 "mask": {"size": window}}
+    out = {"architecture": "Gavipel", "vocab": vocab, "width": width, "norm": {"eps": 1e-5},
+           "embedding": {"scale": float(width) ** 0.5},
+           "layers": [{"type": "attention", "mixer": dict(attention), "mlp": moe} for _ in range(layers)]}
+    if layers >= 3:
+        out["loop"] = {"start": 1, "stop": 3, "times": passes}
+    return out
+
+
+SHAPES["gavipel-w1024"] = gavipel(*COMPARISON_SIZES["w1024"])
+SHAPES["gavipel-w2048"] = gavipel(*COMPARISON_SIZES["w2048"])

@@ -62,10 +62,20 @@ struct TcAttnParams {
                              // the keys of its own chunk up to itself
     float out_scale;         // every result times this
     const float* sinks;      // [n_heads] or null: exp(sink) joins a row's denominator, with no value
+    const __nv_bfloat16* gate;   // rows laid out like `out`, or null: every result times sigmoid(logit)
+    int gate_stride;
     int n_pages;             // of the pool
     int runs;                // 1: the 4-D maps may be used for tiles whose pages are consecutive
     int* status;
 };
+
+// Eight results times the sigmoids of their logits.
+__device__ __forceinline__ void gate_eight(float* o, const __nv_bfloat16* logits) {
+    const uint4 raw = *reinterpret_cast<const uint4*>(logits);
+    const __nv_bfloat16* g = reinterpret_cast<const __nv_bfloat16*>(&raw);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) o[i] *= 1.0f / (1.0f + expf(-__bfloat162float(g[i])));
+}
 
 // HD: the head size, 64 or 128.  Operands whose contracted or free dimension is the head
 // size lie in shared memory as HD / 64 halves of [rows][128 bytes] (one swizzle atom wide).
@@ -591,11 +601,13 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
         const int j_last = group + (my_tiles - 1) * GROUPS;
         if (ok && my_tiles > 0) ok = wait_all(&s.pv_done[j_last % PB], (j_last / PB) & 1);
         __nv_bfloat16* dst = nullptr;
+        const __nv_bfloat16* gate = nullptr;
         float sink = -INFINITY;                       // in the base-2 exponent
         if (real) {
             const int tok = row_base + row / n_rep, head = kv_head * n_rep + row % n_rep;
             if (p.sinks != nullptr) sink = p.sinks[head] * LOG2E;
             dst = p.out + (size_t)tok * p.out_stride + (size_t)head * HD;
+            if (p.gate != nullptr) gate = p.gate + (size_t)tok * p.gate_stride + (size_t)head * HD;
         }
         if (GROUPS > 1) {
             // Two groups: each holds the sums over its own tiles against its own reference.
@@ -632,6 +644,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                                (other_any ? __uint_as_float(b[i]) * w_other : 0.f);
 #pragma unroll
                     for (int q4 = 0; q4 < 4; ++q4) {
+                        if (gate != nullptr) gate_eight(o + 8 * q4, gate + c0 + 8 * q4);
                         uint4 w;
                         w.x = pack_bf16(o[8 * q4 + 0], o[8 * q4 + 1]);
                         w.y = pack_bf16(o[8 * q4 + 2], o[8 * q4 + 3]);
@@ -657,11 +670,15 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                 if (real) {
 #pragma unroll
                     for (int q4 = 0; q4 < 4; ++q4) {
+                        float o[8];
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) o[i] = __uint_as_float(v[8 * q4 + i]) * inv;
+                        if (gate != nullptr) gate_eight(o, gate + c0 + 8 * q4);
                         uint4 w;
-                        w.x = pack_bf16(__uint_as_float(v[8 * q4 + 0]) * inv, __uint_as_float(v[8 * q4 + 1]) * inv);
-                        w.y = pack_bf16(__uint_as_float(v[8 * q4 + 2]) * inv, __uint_as_float(v[8 * q4 + 3]) * inv);
-                        w.z = pack_bf16(__uint_as_float(v[8 * q4 + 4]) * inv, __uint_as_float(v[8 * q4 + 5]) * inv);
-                        w.w = pack_bf16(__uint_as_float(v[8 * q4 + 6]) * inv, __uint_as_float(v[8 * q4 + 7]) * inv);
+                        w.x = pack_bf16(o[0], o[1]);
+                        w.y = pack_bf16(o[2], o[3]);
+                        w.z = pack_bf16(o[4], o[5]);
+                        w.w = pack_bf16(o[6], o[7]);
                         *reinterpret_cast<uint4*>(dst + c0 + 8 * q4) = w;
                     }
                 }
@@ -698,19 +715,21 @@ int launch_as(dim3 grid, cudaStream_t st, const CUtensorMap& mk, const CUtensorM
 // k_cache / v_cache: [n_pages][n_kv_heads][page_tokens][head_dim] bf16; head_dim 64 or 128.
 // keep_first (with a window): a row at position p reads j <= p with p - j < window or j < keep_first.
 // chunked: `window` is a chunk's size (first_key).  sinks: [n_heads] or null.  Results times out_scale.
+// gate: null, or logits laid out like `out`, rows of 16-byte pieces: results times their sigmoids.
 CB_EXPORT int cb_attention_tcgen05_kept(const void* qkv, int qkv_stride, void* out, int out_stride,
                                         const void* k_cache, const void* v_cache, int n_pages,
                                         const int* req_row_start, const int* req_first_pos,
                                         const int* block_table, int table_stride, int n_requests,
                                         int max_new_tokens, int n_heads, int n_kv_heads, int head_dim,
                                         int page_tokens, float scale, int window, int chunked, int keep_first,
-                                        float out_scale, const float* sinks, int lean, int* status, void* stream) {
+                                        float out_scale, const float* sinks, const void* gate, int gate_stride,
+                                        int lean, int* status, void* stream) {
     if (n_requests <= 0 || max_new_tokens <= 0) return 0;
     if (keep_first < 0 || !(scale > 0.f)) return CB_ERR_UNSUPPORTED;
     if ((head_dim != 64 && head_dim != 128) || n_heads % n_kv_heads != 0 || page_tokens < 8 || page_tokens > KEYS ||
         (page_tokens & (page_tokens - 1)) || (qkv_stride & 7) || (out_stride & 7) ||
         ((uintptr_t)qkv & 15) || ((uintptr_t)out & 15) || ((uintptr_t)k_cache & 15) ||
-        ((uintptr_t)v_cache & 15))
+        ((uintptr_t)v_cache & 15) || ((uintptr_t)gate & 15) || (gate != nullptr && (gate_stride & 7)))
         return CB_ERR_UNSUPPORTED;
     int shift = 0;
     while ((1 << shift) < page_tokens) ++shift;
@@ -746,6 +765,8 @@ CB_EXPORT int cb_attention_tcgen05_kept(const void* qkv, int qkv_stride, void* o
     p.keep_first = window > 0 ? keep_first : 0;
     p.chunked = window > 0 && chunked ? 1 : 0;
     p.sinks = sinks;
+    p.gate = (const __nv_bfloat16*)gate;
+    p.gate_stride = gate_stride;
     p.out_scale = out_scale;
     p.status = status;
     const int n_rep = n_heads / n_kv_heads;
@@ -773,5 +794,6 @@ CB_EXPORT int cb_attention_tcgen05(const void* qkv, int qkv_stride, void* out, i
                                    void* stream) {
     return cb_attention_tcgen05_kept(qkv, qkv_stride, out, out_stride, k_cache, v_cache, n_pages, req_row_start,
                                      req_first_pos, block_table, table_stride, n_requests, max_new_tokens, n_heads,
-                                     n_kv_heads, head_dim, page_tokens, scale, window, 0, 0, 1.0f, nullptr, lean, status, stream);
+                                     n_kv_heads, head_dim, page_tokens, scale, window, 0, 0, 1.0f, nullptr, nullptr, 0, lean,
+                                     status, stream);
 }

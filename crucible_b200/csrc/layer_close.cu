@@ -126,7 +126,7 @@ __device__ __forceinline__ void norm_piece(const CloseArgs& a, int t, int i, con
 
 // PER: pieces of V columns that a thread keeps between the two passes (0: any number, read again).
 template <typename T, int V, int PER>
-__global__ void __launch_bounds__(1024) layer_close_kernel(CloseArgs a) {
+__global__ void __launch_bounds__(PER > 0 ? 512 : 1024) layer_close_kernel(CloseArgs a) {
     cb_pdl_trigger();
     cb_pdl_wait();
     __shared__ float scratch[32];
@@ -171,7 +171,7 @@ int launch_close(const CloseArgs& a, int n_rows, bool vec, cudaStream_t s) {
     auto threads = [](int n) { return n < 32 ? 32 : (n + 31) / 32 * 32; };
     if (vec && n4 <= 256) cb_launch(layer_close_kernel<T, 4, 1>, dim3(n_rows), dim3(threads(n4)), 0, s, a);
     else if (vec && n4 <= 512) cb_launch(layer_close_kernel<T, 4, 2>, dim3(n_rows), dim3(threads((n4 + 1) / 2)), 0, s, a);
-    else if (vec && n4 <= 4096) cb_launch(layer_close_kernel<T, 4, 4>, dim3(n_rows), dim3(threads((n4 + 3) / 4)), 0, s, a);
+    else if (vec && n4 <= 2048) cb_launch(layer_close_kernel<T, 4, 4>, dim3(n_rows), dim3(threads((n4 + 3) / 4)), 0, s, a);
     else if (vec) cb_launch(layer_close_kernel<T, 4, 0>, dim3(n_rows), dim3(1024), 0, s, a);
     else cb_launch(layer_close_kernel<T, 1, 0>, dim3(n_rows), dim3(a.width >= 1024 ? 256 : 128), 0, s, a);
     return cb_last_error();

@@ -19,7 +19,7 @@
 //            pair's result does not depend on which other pairs share its tile.
 //   combine  residual[t] += the token's pairs in the order of its choices (or, for the tensor
 //            cores' grouped products, the token's rows of the sorted order times their weights),
-//            and a shared expert's row times the token's gate if it was run apart.
+//            and a shared expert's row times the token's gate (or as it is) if it was run apart.
 #define CB_PDL_BIT 13      // this file's bit in CRUCIBLE_PDL
 #include "common.cuh"
 
@@ -438,7 +438,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ rows, int top, floa
             if (offsets == nullptr) add(rows + p * width + i, 1.0f);
             else add(rows + (size_t)(offsets[idx[p]] + place[p]) * width + i, weight[p]);
         }
-        if (shared != nullptr) add(shared + (size_t)t * width + i, gate[t]);
+        if (shared != nullptr) add(shared + (size_t)t * width + i, gate != nullptr ? gate[t] : 1.0f);
         float* dst = residual + (size_t)t * width + i;
 #pragma unroll
         for (int e = 0; e < V; ++e) dst[e] += sum[e];
@@ -550,7 +550,7 @@ CB_EXPORT int cb_moe_rows_small(int gated, const void* a, int a_stride, const vo
 }
 
 // plan null: rows [tokens * top][width] by pair, weighted; else rows in the sorted order of that plan.
-// shared (or null): rows [tokens][width] that join with gate[token].
+// shared (or null): rows [tokens][width] that join with gate[token] (null: as they are).
 CB_EXPORT int cb_moe_combine(const float* rows, int top, float* residual, int n_tokens, int width,
                              const int* plan, const int* idx, const int* place, const float* weight,
                              const float* shared, const float* gate, void* stream) {

@@ -1,7 +1,7 @@
 // Paged softmax attention whose window keeps the first tokens and whose denominator
-// may hold a learned sink.  Two kernels (the preparation in two forms: the one described
-// first, and a general one with an RMS norm of q and k, either pairing of the rotation and
-// values cached as they are).
+// may hold a learned sink.  Two kernels (the preparation in three forms: the one described
+// first, a general one with an RMS norm of q and k, either pairing of the rotation and
+// values cached as they are, and a quicker one for neighbouring pairs).
 //
 // (1) Preparation of a step's rows, one block per token.  A row of the joint
 //     projection is [q: H*D | k: G*D | v: G*E | ...].  Pairs (2i, 2i+1), i < R/2, of
@@ -208,6 +208,113 @@ __global__ void norm_rotate_append_kernel(T* __restrict__ proj, int proj_stride,
     }
 }
 
+// The same for neighbouring pairs, head by head norms (or none) and values as they are: a lane keeps
+// whole pairs (2p, 2p + 1), p = lane + 32 i, of a head in registers, the angles of its pairs are taken
+// once for all the heads its warp works on, and the next head's row is on its way while one is turned.
+// Sizes even, rows at even offsets.  NP: pairs a lane holds.
+template <typename T> struct PairOf;
+template <> struct PairOf<float> {
+    using Raw = float2;
+    static __device__ __forceinline__ float2 open(const Raw& r) { return r; }
+    static __device__ __forceinline__ Raw pack(float a, float b) { return make_float2(a, b); }
+};
+template <> struct PairOf<__nv_bfloat16> {
+    using Raw = __nv_bfloat162;
+    static __device__ __forceinline__ float2 open(const Raw& r) { return __bfloat1622float2(r); }
+    static __device__ __forceinline__ Raw pack(float a, float b) { return __floats2bfloat162_rn(a, b); }
+};
+
+template <typename T, int NP>
+__global__ void pairs_append_kernel(T* __restrict__ proj, int proj_stride, const float* __restrict__ q_gain,
+                                    const float* __restrict__ k_gain, float qk_eps,
+                                    const float* __restrict__ freq, int rotary_dim,
+                                    const int* __restrict__ positions, const int* __restrict__ row_request,
+                                    const int* __restrict__ block_table, int table_stride,
+                                    T* __restrict__ k_cache, T* __restrict__ v_cache, int n_heads,
+                                    int n_kv_heads, int key_dim, int value_dim, int page_tokens,
+                                    int write_cache) {
+    cb_pdl_trigger();
+    cb_pdl_wait();
+    using P = PairOf<T>;
+    using Raw = typename P::Raw;
+    const int t = blockIdx.x;
+    T* row = proj + (size_t)t * proj_stride;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n_warps = blockDim.x >> 5;
+    const int n_turn = n_heads + (write_cache ? n_kv_heads : 0);
+    const int n_units = n_turn + (write_cache ? n_kv_heads : 0);      // then the heads of values
+    auto source = [&](int u) {
+        return u < n_turn ? row + (size_t)u * key_dim
+                          : row + (size_t)n_turn * key_dim + (size_t)(u - n_turn) * value_dim;
+    };
+    Raw ahead[NP];
+    auto fetch = [&](int u) {
+        const Raw* src = reinterpret_cast<const Raw*>(source(u));
+        const int n = (u < n_turn ? key_dim : value_dim) >> 1;
+#pragma unroll
+        for (int i = 0; i < NP; ++i)
+            if (lane + 32 * i < n) ahead[i] = src[lane + 32 * i];
+    };
+    if (warp < n_units) fetch(warp);
+    const int pos = positions[t], half = rotary_dim >> 1;
+    size_t slot = 0;          // (page, place in it) of this token, in units of one head's tokens
+    if (write_cache) {
+        const int page = block_table[(size_t)row_request[t] * table_stride + pos / page_tokens];
+        slot = (size_t)page * n_kv_heads * page_tokens + pos % page_tokens;
+    }
+    float sn[NP], cs[NP];
+#pragma unroll
+    for (int i = 0; i < NP; ++i) {
+        const int p = lane + 32 * i;
+        sn[i] = 0.f;
+        cs[i] = 1.f;
+        if (p < half) sincosf((float)pos * freq[p], &sn[i], &cs[i]);
+    }
+    for (int u = warp; u < n_units; u += n_warps) {
+        Raw raw[NP];
+#pragma unroll
+        for (int i = 0; i < NP; ++i) raw[i] = ahead[i];
+        if (u + n_warps < n_units) fetch(u + n_warps);
+        if (u >= n_turn) {
+            Raw* dst = reinterpret_cast<Raw*>(v_cache + (slot + (size_t)(u - n_turn) * page_tokens) * value_dim);
+#pragma unroll
+            for (int i = 0; i < NP; ++i)
+                if (lane + 32 * i < (value_dim >> 1)) dst[lane + 32 * i] = raw[i];
+            continue;
+        }
+        const bool is_q = u < n_heads;
+        const float* gain = is_q ? q_gain : k_gain;
+        float2 x[NP];
+        float ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            x[i] = make_float2(0.f, 0.f);
+            if (lane + 32 * i < (key_dim >> 1)) x[i] = P::open(raw[i]);
+            ss = fmaf(x[i].x, x[i].x, ss);
+            ss = fmaf(x[i].y, x[i].y, ss);
+        }
+        if (gain != nullptr) {
+            const float r = 1.0f / sqrtf(cb_warp_sum(ss) / (float)key_dim + qk_eps);
+#pragma unroll
+            for (int i = 0; i < NP; ++i) {
+                const int p = lane + 32 * i;
+                if (p < (key_dim >> 1)) {
+                    x[i].x = x[i].x * r * gain[2 * p];
+                    x[i].y = x[i].y * r * gain[2 * p + 1];
+                }
+            }
+        }
+        Raw* dst = reinterpret_cast<Raw*>(
+            is_q ? row + (size_t)u * key_dim : k_cache + (slot + (size_t)(u - n_heads) * page_tokens) * key_dim);
+#pragma unroll
+        for (int i = 0; i < NP; ++i) {
+            const int p = lane + 32 * i;
+            if (p >= (key_dim >> 1)) continue;
+            dst[p] = p < half ? P::pack(x[i].x * cs[i] - x[i].y * sn[i], x[i].y * cs[i] + x[i].x * sn[i])
+                              : P::pack(x[i].x, x[i].y);
+        }
+    }
+}
+
 template <typename T, int MAX_PER_LANE>
 __global__ void sink_attention_kernel(
     const T* __restrict__ q, int q_stride, const T* __restrict__ gate, int gate_stride,
@@ -325,6 +432,33 @@ CB_EXPORT int cb_norm_rotate_append(void* proj, int proj_stride, int dtype, cons
                                     int write_cache, float value_eps, int whole_norm, void* stream) {
     if (n_rows <= 0) return 0;
     if (rotary_dim < 0 || rotary_dim > key_dim || (rotary_dim & 1) || key_dim > 4096) return CB_ERR_UNSUPPORTED;
+    const int elem = dtype == CB_F32 ? 4 : 2;
+    const bool pairs = !split_halves && !whole_norm && value_eps < 0.f && !(key_dim & 1) && !(value_dim & 1) &&
+                       !(proj_stride & 1) && key_dim <= 512 && value_dim <= 512 &&
+                       (((uintptr_t)proj | (uintptr_t)k_cache | (uintptr_t)v_cache) & (2 * elem - 1)) == 0;
+    if (pairs) {
+        // few tokens: a warp for every head; many: blocks of warps that take several heads in turn
+        const int units = n_heads + (write_cache ? 2 * n_kv_heads : 0), most = n_rows <= 128 ? 16 : 4;
+        const dim3 block(32 * (units > most ? most : units));
+        const int np = ((key_dim > value_dim ? key_dim : value_dim) + 63) / 64;
+        cudaStream_t st = (cudaStream_t)stream;
+#define CB_PAIRS(TT, NN)                                                                                       \
+    cb_launch(pairs_append_kernel<TT, NN>, dim3(n_rows), block, 0, st, (TT*)proj, proj_stride, q_gain, k_gain, \
+              qk_eps, freq, rotary_dim, positions, row_request, block_table, table_stride, (TT*)k_cache,       \
+              (TT*)v_cache, n_heads, n_kv_heads, key_dim, value_dim, page_tokens, write_cache)
+#define CB_PAIRS_OF(TT)                                                                                        \
+    do {                                                                                                       \
+        if (np == 1) CB_PAIRS(TT, 1);                                                                          \
+        else if (np == 2) CB_PAIRS(TT, 2);                                                                     \
+        else if (np <= 4) CB_PAIRS(TT, 4);                                                                     \
+        else CB_PAIRS(TT, 8);                                                                                  \
+    } while (0)
+        if (dtype == CB_F32) CB_PAIRS_OF(float);
+        else CB_PAIRS_OF(__nv_bfloat16);
+#undef CB_PAIRS_OF
+#undef CB_PAIRS
+        return cb_last_error();
+    }
     int warps = n_heads + n_kv_heads;
     warps = warps > 8 ? 8 : warps;
     const size_t smem = ((size_t)warps * key_dim + 2 * warps) * sizeof(float);

@@ -113,13 +113,14 @@ def expert_rows_small(gated: bool, a, w, n_out: int, plan, n_experts: int, tiles
 def combine(rows, top: int, residual, by_plan=None, shared=None, gate=None) -> None:
     """residual[t] += sum over the token's choices, in their order.  `rows` lie pair by pair and
     weighted, or, with `by_plan` = (plan, idx, place, weight) of `route`, in the sorted order and are
-    weighted here.  `shared` (float32 rows by token) joins with `gate` (float32 [tokens])."""
+    weighted here.  `shared` (float32 rows by token) joins with `gate` (float32
+    [tokens]; None: as it is)."""
     plan, idx, place, weight = by_plan if by_plan is not None else (None,) * 4
     _need_cuda(rows, residual, plan, idx, place, weight, shared, gate)
     if (rows.dtype != torch.float32 or residual.dtype != torch.float32 or not residual.is_contiguous()
-            or not rows.is_contiguous() or (shared is None) != (gate is None)
+            or not rows.is_contiguous() or (shared is None and gate is not None)
             or (shared is not None and (shared.dtype != torch.float32 or shared.shape != residual.shape
-                                        or not shared.is_contiguous() or gate.dtype != torch.float32))):
+                                        or not shared.is_contiguous() or (gate is not None and gate.dtype != torch.float32)))):
         raise KernelError("moe combine adds float32 rows into the float32 residual")
     lib = build.load("moe")
     _check(lib.cb_moe_combine(_ptr(rows), _c_int(top), _ptr(residual), _c_int(residual.shape[0]),

@@ -116,7 +116,7 @@ def _tensor_cores(q, gate, out, sinks, n_heads, n_kv_heads, key_dim, value_dim, 
                   keep_first, out_scale, ctx, cache, k_cache, v_cache, table, gate_per_head=False,
                   chunked=False) -> bool:
     """For bfloat16 rows: steps of prompts' portions alone whose keys and values have one size, 64
-    or 128, without a gate per feature take the tcgen05 attention (`csrc/attention_tcgen05.cu`);
+    or 128, take the tcgen05 attention (`csrc/attention_tcgen05.cu`);
     everything else of key and value sizes that are multiples of 16 up to 256 the mma.sync kernel of 64-row
     tiles (`csrc/attention_mma.cu`, its extended form): prompts' portions and decoded tokens in
     one launch, the rows of a request's query heads that share a key/value head packed into
@@ -129,11 +129,12 @@ def _tensor_cores(q, gate, out, sinks, n_heads, n_kv_heads, key_dim, value_dim, 
     from . import tensor_core
     # keys and values of 64 or 128 features, portions of prompts only: the tcgen05 attention, whose
     # tiles take the kept first tokens ahead of the window's
-    if (key_dim == value_dim and (gate is None or gate_per_head)
+    if (key_dim == value_dim
             and tensor_core.prompt_attention(q, out, k_cache, v_cache, n_heads, n_kv_heads, key_dim, scale,
                                              window, keep_first, ctx, cache, table, chunked=chunked, sinks=sinks,
-                                             out_scale=out_scale)):
-        if gate is not None:
+                                             out_scale=out_scale,
+                                             gate=None if gate_per_head else gate)):
+        if gate is not None and gate_per_head:
             # one logit a head: a pass over the heads' results behind the attention
             from . import latent
             latent.head_gate(out, gate, n_heads, value_dim)

@@ -494,10 +494,12 @@ class _Requests:
 
 
 def _attention_tcgen05(qkv, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, head_dim, scale,
-                       window, cache, keep_first: int = 0, chunked: bool = False, sinks=None, out_scale: float = 1.0) -> bool:
+                       window, cache, keep_first: int = 0, chunked: bool = False, sinks=None, out_scale: float = 1.0,
+                       gate=None) -> bool:
     """tcgen05 attention for portions of prompts: head size 64 or 128, page size a
     power of two from 8 to 128.  `keep_first` (with a window): keys before that position stay
     visible.  `chunked`: the window is a chunk's size.  `sinks`: float32 per query head or None.
+    `gate`: rows laid out like `out` whose sigmoids the results are multiplied by, or None.
     Returns False for anything else."""
     pt = cache.page_tokens
     if pt < 8 or pt > 128 or pt & (pt - 1):
@@ -511,7 +513,9 @@ def _attention_tcgen05(qkv, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, he
         _c_int(reqs.table_stride), _c_int(reqs.count), _c_int(reqs.max_new),
         _c_int(n_heads), _c_int(n_kv_heads), _c_int(head_dim), _c_int(pt),
         ctypes.c_float(scale), _c_int(window or 0), _c_int(1 if chunked else 0), _c_int(keep_first if window else 0),
-        ctypes.c_float(out_scale), _c_void_p(sinks.data_ptr() if sinks is not None else 0), _c_int(ATTENTION_LEAN), _c_void_p(status_word(qkv.device).data_ptr()), _stream())
+        ctypes.c_float(out_scale), _c_void_p(sinks.data_ptr() if sinks is not None else 0),
+        _c_void_p(gate.data_ptr() if gate is not None else 0), _c_int(gate.stride(0) if gate is not None else 0),
+        _c_int(ATTENTION_LEAN), _c_void_p(status_word(qkv.device).data_ptr()), _stream())
     if code == _UNSUPPORTED:
         return False
     if code != 0:
@@ -615,21 +619,23 @@ def wide_row_chunk_keys(blocks_per_chunk: int, context_bucket: int, window) -> i
 
 
 def prompt_attention(q, out, k_cache, v_cache, n_heads, n_kv_heads, head_dim, scale, window, keep_first,
-                     ctx, cache, table, chunked: bool = False, sinks=None, out_scale: float = 1.0) -> bool:
+                     ctx, cache, table, chunked: bool = False, sinks=None, out_scale: float = 1.0,
+                     gate=None) -> bool:
     """The tcgen05 attention for a step that holds portions of prompts only (no single decoded
     tokens ahead of them) over keys and values of one size, 64 or 128, with a window that may
     keep the first tokens or (`chunked`) is the size of chunks, and with a sink per head in the
-    softmax (`sinks`) or none; no gate.  `q`: rows of n_heads * head_dim.  False: not taken."""
+    softmax (`sinks`) or none; `gate`: a logit for every result, or None.  `q`: rows of n_heads * head_dim.  False: not taken."""
     host = getattr(ctx, "host", None)
     n_rep = n_heads // n_kv_heads
     if (not USE_TCGEN05_ATTENTION or host is None or q.dtype != torch.bfloat16 or head_dim not in (64, 128)
             or k_cache.dtype != torch.bfloat16 or host.lead_single != 0 or host.max_new_tokens * n_rep < 64
             or q.stride(0) % 8 or out.stride(0) % 8 or q.data_ptr() % 16 or out.data_ptr() % 16
+            or (gate is not None and (gate.dtype != q.dtype or gate.stride(0) % 8 or gate.data_ptr() % 16))
             or k_cache.shape[-1] != head_dim or v_cache.shape[-1] != head_dim):
         return False
     reqs = _Requests(ctx, table, 0, ctx.n_requests, host.max_new_tokens, host.context_bucket, ctx.n_tokens)
     return _attention_tcgen05(q, out, k_cache, v_cache, reqs, n_heads, n_kv_heads, head_dim, scale, window, cache,
-                              keep_first=keep_first, chunked=chunked, sinks=sinks, out_scale=out_scale)
+                              keep_first=keep_first, chunked=chunked, sinks=sinks, out_scale=out_scale, gate=gate)
 
 
 SPLIT_ROWS = 16          # packed rows (new tokens x heads of a group) the split form takes

@@ -116,7 +116,7 @@ class SinkWindowAttention(BranchMixer):
         cache = ctx.cache(binding.group)
         freq, rotary_dim = (self.position.frequencies() if self.position is not None else (None, 0))
         split = bool(getattr(self.position, "split_halves", False))
-        if self.qk_eps is None and not split:
+        if self.qk_eps is None and not split and self.value_eps is not None:
             kernels.rotate_norm_append(proj, freq, rotary_dim, s.n_heads, s.n_kv_heads, s.head_dim,
                                        self.value_dim, self.value_eps, ctx, cache, binding)
         else:

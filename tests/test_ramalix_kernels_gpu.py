@@ -459,6 +459,6 @@ def test_groups_of_experts_in_the_routing_kernel():
     for i, chosen in enumerate([[0, 4, 5], [0, 1, 2], [2, 5, 4]]):
         assert torch.allclose(wt[i, :3], 0.5 * torch.softmax(logits[i, chosen].cpu(), -1))
     assert count.tolist() == [0] * (n + ns) and sorted(order.tolist()) == list(range(pairs))
-    for bad in ({"groups": (4, 2)}, {"groups": (3, 1)}, {"groups": (3, 4)}, {"n_shared": 1, "gate_col": -1}):
+    for bad in ({"groups": (4, 2)}, {"groups": (3, 1)}, {"groups": (3, 4)}):
         with pytest.raises(k.KernelError):
             k.route(logits, top, idx, weight, place, count, plan, tiles, order, n_experts=n, **bad)
